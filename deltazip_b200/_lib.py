@@ -30,6 +30,8 @@ DZ_DTYPE_BF16 = 1
 DZ_DTYPE_F32 = 2
 DZ_INDEX_I32 = 0
 DZ_INDEX_I64 = 1
+DZ_ACT_SILU = 0
+DZ_ACT_GELU_TANH = 1
 DZ_SBMM_ACCUMULATE = 1
 DZ_SBMM_INPUTS_STABLE = 2
 
@@ -53,6 +55,32 @@ class SbmmArgs(Structure):
         ("workspace", c_void_p), ("workspace_bytes", c_size_t),
         ("y_stride", c_int64),
         ("push", POINTER(PushTarget)),
+    ]
+
+
+class WindowAttentionArgs(Structure):
+    """Mirror of dz_window_attention_args."""
+    _fields_ = [
+        ("qkv", c_void_p), ("row_stride", c_int64), ("k_off", c_int32), ("v_off", c_int32), ("out", c_void_p),
+        ("k_cache", c_void_p), ("v_cache", c_void_p), ("block_tables", c_void_p),
+        ("ring_blocks", c_int32), ("block_size", c_int32), ("q_starts", c_void_p), ("ctx_lens", c_void_p),
+        ("num_seqs", c_int32), ("rows", c_int32), ("max_q", c_int32), ("decode", c_int32),
+        ("heads", c_int32), ("kv_heads", c_int32), ("dim", c_int32), ("vdim", c_int32),
+        ("scale", c_float), ("window", c_int32), ("bias", c_void_p), ("bias_len", c_int32), ("splits", c_int32),
+        ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("dtype", c_int32),
+    ]
+
+
+class MlstmArgs(Structure):
+    """Mirror of dz_mlstm_args."""
+    _fields_ = [
+        ("x", c_void_p), ("row_stride", c_int64), ("k_off", c_int32), ("v_off", c_int32), ("g_off", c_int32),
+        ("h", c_void_p), ("w_if", c_void_p), ("b_if", c_void_p), ("pre_if", c_void_p), ("width", c_int32),
+        ("cap", c_float), ("scale", c_float), ("norm_weight", c_void_p), ("eps", c_float), ("out", c_void_p),
+        ("S", c_void_p), ("n", c_void_p), ("m", c_void_p), ("slots", c_void_p), ("q_starts", c_void_p),
+        ("ctx_lens", c_void_p), ("num_seqs", c_int32), ("rows", c_int32), ("heads", c_int32), ("dim", c_int32),
+        ("vdim", c_int32), ("chunkwise", c_int32), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
+        ("dtype", c_int32),
     ]
 
 
@@ -103,6 +131,20 @@ _SIGNATURES = {
     "dz_paged_attention_decode": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                                           c_void_p, c_size_t, c_int, c_void_p]),
+    "dz_embed_norm": (c_int, [c_void_p, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p, c_int64, c_int,
+                              c_int, c_float, c_int, c_void_p]),
+    "dz_residual_norm": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int64,
+                                 c_int, c_int, c_float, c_int, c_void_p]),
+    "dz_gated_act": (c_int, [c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "dz_qk_norm": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
+                           c_void_p, c_int, c_int, c_void_p]),
+    "dz_kv_append": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                             c_void_p]),
+    "dz_window_attention_workspace_bytes": (c_size_t, [c_int, c_int, c_int, c_int, c_int]),
+    "dz_window_attention": (c_int, [POINTER(WindowAttentionArgs), c_void_p]),
+    "dz_mlstm_chunk_supported": (c_int, [c_int, c_int, c_int]),
+    "dz_mlstm_workspace_bytes": (c_size_t, [c_int, c_int]),
+    "dz_mlstm": (c_int, [POINTER(MlstmArgs), c_void_p]),
     "dz_slot_upload": (c_int, [c_void_p, c_void_p, c_size_t, c_int, c_void_p]),
     "dz_slot_reset": (c_int, [c_void_p, c_size_t, c_void_p]),
     "dz_stream_fence": (c_int, [c_void_p]),

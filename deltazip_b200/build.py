@@ -45,7 +45,7 @@ def _digest() -> str:
         os.path.join(PKG_DIR, "..", "include", "deltazip_b200.h"), os.path.abspath(__file__)]
     for f in files:
         with open(f, "rb") as fh:
-            h.update(f.encode())
+            h.update(os.path.basename(f).encode())      # not the path: a built tree may be moved
             h.update(fh.read())
     return h.hexdigest()
 
@@ -71,10 +71,12 @@ def build_library(force: bool = False, verbose: bool = False) -> str:
         if p.returncode != 0:
             raise RuntimeError(f"nvcc failed on {src}:\n{out}")
         objs.append(obj)
-    cmd = [_nvcc(), "-shared", "-o", LIB_PATH, *objs, "-lcudart_static", "-ldl", "-lrt", "-lpthread"]
+    part = f"{LIB_PATH}.{os.getpid()}"
+    cmd = [_nvcc(), "-shared", "-o", part, *objs, "-lcudart_static", "-ldl", "-lrt", "-lpthread"]
     out = subprocess.run(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)
     if out.returncode != 0:
         raise RuntimeError("link failed:\n" + out.stdout)
+    os.replace(part, LIB_PATH)                  # a process that has the old library open keeps it
     with open(os.path.join(PKG_DIR, "build", "ptxas.log"), "w") as fh:
         fh.write("\n".join(logs))
     with open(STAMP, "w") as fh:

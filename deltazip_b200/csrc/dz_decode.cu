@@ -9,46 +9,12 @@
 //   paged_attention_v1              ops.h:6       (attention/attention_kernels.cu)
 // Layouts are this library's own: the KV cache is [num_blocks, block_size, kv_heads, 128] for K
 // and for V (one 256-byte row per token and head), head size 128 only (every Llama-2 size).
-#include <cuda_bf16.h>
-#include <cuda_fp16.h>
-#include <math.h>
-
-#include "dz_common.cuh"
+#include "dz_elem.cuh"
 
 namespace dz {
 namespace {
 
 constexpr int kHeadDim = 128;
-
-template <typename T> struct Cvt;
-template <> struct Cvt<__half> {
-  static __device__ __forceinline__ float2 up(uint32_t v) {
-    return __half22float2(*reinterpret_cast<const __half2*>(&v));
-  }
-  static __device__ __forceinline__ uint32_t down(float a, float b) {
-    __half2 h = __floats2half2_rn(a, b);
-    return *reinterpret_cast<uint32_t*>(&h);
-  }
-  static __device__ __forceinline__ float round(float a) { return __half2float(__float2half_rn(a)); }
-};
-template <> struct Cvt<__nv_bfloat16> {
-  static __device__ __forceinline__ float2 up(uint32_t v) {
-    return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v));
-  }
-  static __device__ __forceinline__ uint32_t down(float a, float b) {
-    __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<uint32_t*>(&h);
-  }
-  static __device__ __forceinline__ float round(float a) {
-    return __bfloat162float(__float2bfloat16_rn(a));
-  }
-};
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
 
 // ---------------------------------------------------------------------------
 // RMSNorm, optionally preceded by the residual add.  One CTA per token row; the row is read
@@ -438,20 +404,6 @@ paged_decode_attention_kernel(const T* __restrict__ qkv, int q_row_stride, T* __
     }
     out[((size_t)seq * q_heads + head) * kHeadDim + d] = (T)(ll > 0.f ? a / ll : 0.f);
   }
-}
-
-template <typename K, typename... Args>
-cudaError_t launch_pdl(K kern, dim3 grid, dim3 block, cudaStream_t st, Args... args) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = grid;
-  cfg.blockDim = block;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = 1;
-  return cudaLaunchKernelEx(&cfg, kern, args...);
 }
 
 template <typename T>

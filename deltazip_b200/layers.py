@@ -55,13 +55,18 @@ class _ParallelLinearBase(nn.Module):
         return {"weight": self.weight}
 
 
+def _cut(total: int):
+    """This rank's [lo, hi) of a weight dimension: whole 128-wide units, or any size on one rank."""
+    size = get_tensor_model_parallel_world_size()
+    return (0, total) if size == 1 else shard_range(total, SHARD_UNIT, get_tensor_model_parallel_rank(), size)
+
+
 class ColumnParallelLinear(_ParallelLinearBase):
     """y = x W^T with W split along the output dimension (whole 128-row tiles per rank)."""
 
     def __init__(self, input_size: int, output_size: int, full_weight: Optional[torch.Tensor] = None,
                  gather_output: bool = False, device="cuda", dtype=torch.float16):
-        rank, size = get_tensor_model_parallel_rank(), get_tensor_model_parallel_world_size()
-        lo, hi = shard_range(output_size, SHARD_UNIT, rank, size)
+        lo, hi = _cut(output_size)
         if full_weight is None:
             w = torch.empty((hi - lo, input_size), dtype=dtype, device=device).normal_(0, 0.02)
         else:
@@ -82,16 +87,16 @@ class MergedColumnParallelLinear(ColumnParallelLinear):
     def __init__(self, input_size: int, output_sizes: List[int],
                  full_weights: Optional[List[torch.Tensor]] = None, device="cuda",
                  dtype=torch.float16):
-        rank, size = get_tensor_model_parallel_rank(), get_tensor_model_parallel_world_size()
-        parts, self.shards = [], []
+        parts, shards = [], []
         for i, out in enumerate(output_sizes):
-            lo, hi = shard_range(out, SHARD_UNIT, rank, size)
-            self.shards.append((lo, hi))
+            lo, hi = _cut(out)
+            shards.append((lo, hi))
             if full_weights is None:
                 parts.append(torch.empty((hi - lo, input_size), dtype=dtype, device=device).normal_(0, 0.02))
             else:
                 parts.append(full_weights[i][lo:hi].to(device=device, dtype=dtype))
         _ParallelLinearBase.__init__(self, torch.cat(parts, dim=0).contiguous())
+        self.shards = shards
         self.input_size, self.output_sizes = input_size, list(output_sizes)
         self.output_size = sum(output_sizes)
         self.gather_output = False
@@ -120,8 +125,7 @@ class RowParallelLinear(_ParallelLinearBase):
     def __init__(self, input_size: int, output_size: int, full_weight: Optional[torch.Tensor] = None,
                  input_is_parallel: bool = True, reduce_results: bool = True, device="cuda",
                  dtype=torch.float16):
-        rank, size = get_tensor_model_parallel_rank(), get_tensor_model_parallel_world_size()
-        lo, hi = shard_range(input_size, SHARD_UNIT, rank, size)
+        lo, hi = _cut(input_size)
         if full_weight is None:
             w = torch.empty((output_size, hi - lo), dtype=dtype, device=device).normal_(0, 0.02)
         else:

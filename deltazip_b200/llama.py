@@ -13,7 +13,7 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Callable, List, Optional, Sequence
+from typing import Callable, Dict, Optional
 
 import torch
 import torch.nn as nn
@@ -21,6 +21,8 @@ import torch.nn.functional as F
 
 from . import layers as L
 from . import ops
+from .cache import AttnMeta, PagedKVCache  # noqa: F401  (re-exported: callers import them from here)
+from .loader import copy_weights
 from .parallel_state import (SHARD_UNIT, get_tensor_model_parallel_rank,
                              get_tensor_model_parallel_world_size, shard_range)
 
@@ -36,6 +38,13 @@ class LlamaConfig:
     rms_norm_eps: float = 1e-5
     rope_theta: float = 10000.0
 
+    @classmethod
+    def from_dict(cls, d: dict) -> "LlamaConfig":
+        """From a parsed config.json with the usual key names."""
+        keys = ("hidden_size", "intermediate_size", "num_hidden_layers", "num_attention_heads",
+                "num_key_value_heads", "vocab_size", "rms_norm_eps", "rope_theta")
+        return cls(**{k: d[k] for k in keys if d.get(k) is not None})
+
     @property
     def head_dim(self) -> int:
         return self.hidden_size // self.num_attention_heads
@@ -48,46 +57,6 @@ class LlamaConfig:
 LLAMA2_7B = LlamaConfig(4096, 11008, 32, 32, None)
 LLAMA2_13B = LlamaConfig(5120, 13824, 40, 40, None)
 LLAMA2_70B = LlamaConfig(8192, 28672, 80, 64, 8)
-
-
-class PagedKVCache:
-    """Per-layer K and V pools of `num_blocks` blocks of `block_size` tokens, [slots, kv_heads,
-    128] each, with a free list (role of the reference's block manager + cache engine,
-    serving/vllm/core/block_manager.py, serving/vllm/worker/cache_engine.py, reduced to what a
-    single process needs)."""
-
-    def __init__(self, num_layers: int, num_blocks: int, kv_heads: int, block_size: int = 16,
-                 dtype=torch.float16, device="cuda"):
-        self.block_size, self.num_blocks, self.kv_heads = block_size, num_blocks, kv_heads
-        shape = (num_blocks * block_size, kv_heads, 128)
-        self.k = [torch.empty(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.v = [torch.empty(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.free: List[int] = list(range(num_blocks - 1, -1, -1))
-
-    def allocate(self, n_blocks: int) -> List[int]:
-        if n_blocks > len(self.free):
-            raise RuntimeError("out of KV cache blocks")
-        return [self.free.pop() for _ in range(n_blocks)]
-
-    def release(self, blocks: Sequence[int]) -> None:
-        self.free.extend(blocks)
-
-    def slots(self, blocks: Sequence[int], start: int, count: int) -> List[int]:
-        """Cache slots of token positions [start, start + count) of a sequence owning `blocks`."""
-        bs = self.block_size
-        return [blocks[p // bs] * bs + p % bs for p in range(start, start + count)]
-
-
-@dataclass
-class AttnMeta:
-    """How attention runs in one forward pass.  Decode: `block_tables` [B, max_blocks] int32 and
-    `seq_lens` [B] int32 (cached length including the current token).  Prefill: `prompt_lens`,
-    the token count of each sequence, rows in (sequence, position) order."""
-    slot_mapping: Optional[torch.Tensor] = None          # int64 [M] cache slot per token, -1 = none
-    block_tables: Optional[torch.Tensor] = None
-    seq_lens: Optional[torch.Tensor] = None
-    prompt_lens: Optional[List[int]] = None
-    splits: int = 1
 
 
 class LlamaDecoderLayer(nn.Module):
@@ -111,6 +80,7 @@ class LlamaForCausalLM(nn.Module):
     supported_delta_modules = ["qkv_proj", "o_proj", "gate_up_proj", "down_proj"]
     packed_modules_mapping = {"qkv_proj": ["q_proj", "k_proj", "v_proj"],
                               "gate_up_proj": ["gate_proj", "up_proj"]}
+    supports_portions = False           # a prompt runs in one piece: prefill does not read the cache
 
     def __init__(self, cfg: LlamaConfig, device="cuda", seed: int = 0, dtype=torch.float16):
         super().__init__()
@@ -141,6 +111,30 @@ class LlamaForCausalLM(nn.Module):
         del full
         # a custom linear hook lets the same model run the reference's PyTorch path
         self.linear_override: Optional[Callable[[str, nn.Module, torch.Tensor], torch.Tensor]] = None
+
+    def make_cache(self, num_blocks: int, block_size: int, max_seqs: int) -> PagedKVCache:
+        return PagedKVCache(self.cfg.num_hidden_layers, num_blocks, self.kv_heads, block_size, self.dtype,
+                            self.embed_tokens.device)
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        """Copies a checkpoint's tensors (the names of the published Llama checkpoints, which the
+        reference's loader reads, serving/vllm/model_executor/models/llama.py:360-407) into the base
+        layers.  One rank only."""
+        if self.tp_size != 1:
+            raise ValueError("loading a base checkpoint is implemented for one rank")
+        want = {"model.embed_tokens.weight": [self.embed_tokens], "model.norm.weight": [self.norm],
+                "lm_head.weight": [self.lm_head]}
+        for i, layer in enumerate(self.layers):
+            pre = f"model.layers.{i}."
+            want[pre + "input_layernorm.weight"] = [layer.input_layernorm]
+            want[pre + "post_attention_layernorm.weight"] = [layer.post_attention_layernorm]
+            for module, names in ((layer.qkv_proj, ("q", "k", "v")), (layer.gate_up_proj, ("gate", "up"))):
+                parts = module.weight.split([hi - lo for lo, hi in module.shards])
+                sub = "self_attn." if len(names) == 3 else "mlp."
+                want.update({f"{pre}{sub}{n}_proj.weight": [part] for n, part in zip(names, parts)})
+            want[pre + "self_attn.o_proj.weight"] = [layer.o_proj.weight]
+            want[pre + "mlp.down_proj.weight"] = [layer.down_proj.weight]
+        copy_weights(want, tensors)
 
     def _linear(self, name: str, module: nn.Module, x: torch.Tensor) -> torch.Tensor:
         if self.linear_override is not None:

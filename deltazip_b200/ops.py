@@ -313,14 +313,14 @@ def stream_fence() -> None:
 def base_gemm(x: torch.Tensor, base_weight: torch.Tensor,
               out: Optional[torch.Tensor] = None, stable: bool = False) -> torch.Tensor:
     """y = x W^T on the same kernel (every token base-only); the library GEMM for more than
-    FUSED_MAX_TOKENS rows."""
+    FUSED_MAX_TOKENS rows, for shapes the kernel does not tile and for 32-bit activations."""
     _need_cuda(x, base_weight)
     x2 = x.reshape(-1, x.shape[-1])
     if not x2.is_contiguous():
         x2 = x2.contiguous()
     m, k = x2.shape
     n = base_weight.shape[0]
-    if m > FUSED_MAX_TOKENS:
+    if m > FUSED_MAX_TOKENS or n % 128 or k % 64 or x.dtype == torch.float32:
         if out is None:
             return torch.matmul(x2, base_weight.t()).reshape(*x.shape[:-1], n)
         torch.matmul(x2, base_weight.t(), out=out.reshape(m, n))
@@ -603,4 +603,171 @@ def paged_attention_decode(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: to
         block_tables.data_ptr(), block_tables.shape[1], seq_lens.data_ptr(), b, q_heads, kv_heads,
         128, block_size, float(scale), splits, ws_ptr, ws_bytes, _dtype_code(qkv), _stream()),
         "dz_paged_attention_decode")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# decoder steps with a 32-bit residual stream, sliding-window attention over a ring of cache
+# blocks, matrix-memory recurrence.  16-bit or 32-bit activations, any sizes.
+# ---------------------------------------------------------------------------
+
+ACTIVATIONS = {"silu": _lib.DZ_ACT_SILU, "gelu_tanh": _lib.DZ_ACT_GELU_TANH}
+_scratch = {}
+
+
+def _zeroed_scratch(kind: str, device, nbytes: int) -> Optional[torch.Tensor]:
+    """Grow-only scratch per (kernel, device, stream), zero-filled when it is made: the kernels
+    leave their tickets at zero."""
+    if nbytes == 0:
+        return None
+    key = (kind, device.index, _stream())
+    buf = _scratch.get(key)
+    if buf is None or buf.numel() < nbytes:
+        buf = torch.zeros(nbytes, dtype=torch.uint8, device=device)
+        _scratch[key] = buf
+    return buf
+
+
+def _any_dtype_code(t: torch.Tensor) -> int:
+    return _lib.DZ_DTYPE_F32 if t.dtype == torch.float32 else _dtype_code(t)
+
+
+def _ptr(t: Optional[torch.Tensor]):
+    return None if t is None else t.data_ptr()
+
+
+def matmul_f32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """x W^T with a 32-bit result (library GEMM, 32-bit accumulation)."""
+    _need_cuda(x, weight)
+    if x.dtype == torch.float32:
+        return torch.mm(x, weight.t())
+    return torch.mm(x, weight.t(), out_dtype=torch.float32)
+
+
+def embed_norm(tokens: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float, weight_offset: float = 0.0,
+               copy: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """norm(table[tokens]) as a 32-bit residual [M, width]; `copy`: a column slice of a wider matrix
+    that gets the same rounded to the table's type."""
+    _need_cuda(tokens, table, weight, copy)
+    m, (vocab, width) = tokens.numel(), table.shape
+    residual = torch.empty((m, width), dtype=torch.float32, device=table.device)
+    if copy is not None and (copy.dtype != table.dtype or copy.shape != (m, width) or copy.stride(1) != 1):
+        raise ValueError("copy must be a [tokens, width] slice of the table's type with unit column stride")
+    check(lib().dz_embed_norm(tokens.data_ptr(), table.data_ptr(), vocab, weight.data_ptr(), float(weight_offset),
+                              residual.data_ptr(), _ptr(copy), copy.stride(0) if copy is not None else 0, m, width,
+                              float(eps), _any_dtype_code(table), _stream()), "dz_embed_norm")
+    return residual
+
+
+def residual_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float,
+                  dtype: torch.dtype, weight_offset: float = 0.0, vec: Optional[torch.Tensor] = None,
+                  replace: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """residual (32-bit, in place) += delta + vec, or = with `replace`; returns norm(residual) in
+    `dtype`, or the residual rounded to it when `weight` is None."""
+    _need_cuda(residual, delta, weight, vec, out)
+    m, width = residual.shape
+    if out is None:
+        out = torch.empty((m, width), dtype=dtype, device=residual.device)
+    if residual.dtype != torch.float32 or not residual.is_contiguous() or out.stride(1) != 1:
+        raise ValueError("the residual is a contiguous float32 matrix, out has unit column stride")
+    if delta is not None and (delta.shape != residual.shape or not delta.is_contiguous()):
+        raise ValueError("delta must be a contiguous matrix of the residual's shape")
+    check(lib().dz_residual_norm(residual.data_ptr(), _ptr(delta), _any_dtype_code(delta) if delta is not None else 0,
+                                 int(replace), _ptr(vec), _ptr(weight), float(weight_offset), out.data_ptr(),
+                                 out.stride(0) if m > 1 else max(out.stride(0), width), m, width, float(eps),
+                                 _any_dtype_code(out), _stream()), "dz_residual_norm")
+    return out
+
+
+def gated_act(x: torch.Tensor, activation: str, inter: Optional[int] = None) -> torch.Tensor:
+    """act(x[:, :inter]) * x[:, inter:2 inter]; columns beyond are padding."""
+    _need_cuda(x)
+    inter = inter or x.shape[1] // 2
+    out = torch.empty((x.shape[0], inter), dtype=x.dtype, device=x.device)
+    check(lib().dz_gated_act(x.data_ptr(), x.stride(0), out.data_ptr(), x.shape[0], inter, ACTIVATIONS[activation],
+                             _any_dtype_code(x), _stream()), "dz_gated_act")
+    return out
+
+
+def qk_norm(qkv: torch.Tensor, wq: torch.Tensor, wk: torch.Tensor, v_width: int, eps: float,
+            k_cache: Optional[torch.Tensor] = None, v_cache: Optional[torch.Tensor] = None,
+            slot_mapping: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMS norm of the query row and of the key row of [q | k | v | ...] rows in place (each over all
+    its heads); with `slot_mapping` the key and value also go to the cache."""
+    _need_cuda(qkv, wq, wk, k_cache, v_cache, slot_mapping)
+    check(lib().dz_qk_norm(qkv.data_ptr(), qkv.stride(0), wq.numel(), wk.numel(), v_width, wq.data_ptr(),
+                           wk.data_ptr(), float(eps), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), qkv.shape[0],
+                           _any_dtype_code(qkv), _stream()), "dz_qk_norm")
+    return qkv
+
+
+def kv_append(qkv: torch.Tensor, k_off: int, k_cache: torch.Tensor, v_cache: torch.Tensor,
+              slot_mapping: torch.Tensor) -> None:
+    """Copies the key and value parts of every row to its cache slot (< 0: not kept)."""
+    _need_cuda(qkv, k_cache, v_cache, slot_mapping)
+    check(lib().dz_kv_append(qkv.data_ptr(), qkv.stride(0), k_off, k_cache[0].numel(), v_cache[0].numel(),
+                             k_cache.data_ptr(), v_cache.data_ptr(), slot_mapping.data_ptr(), qkv.shape[0],
+                             _any_dtype_code(qkv), _stream()), "dz_kv_append")
+
+
+def window_attention(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor,
+                     q_starts: torch.Tensor, ctx_lens: torch.Tensor, max_query: int, decode: bool, heads: int,
+                     block_size: int, scale: float, window: int, bias: Optional[torch.Tensor] = None,
+                     splits: int = 0) -> torch.Tensor:
+    """Attention of [q | k | v | ...] rows with a sliding window and an additive bias per distance
+    ([heads, distances] float32); see dz_window_attention.  `splits` 0: enough CTAs to fill the GPU."""
+    _need_cuda(qkv, k_cache, v_cache, block_tables, q_starts, ctx_lens, bias)
+    kv_heads, dim, vdim = k_cache.shape[1], k_cache.shape[2], v_cache.shape[2]
+    rows, seqs = qkv.shape[0], ctx_lens.shape[0]
+    if any(t.dtype != torch.int32 or not t.is_contiguous() for t in (block_tables, q_starts, ctx_lens)):
+        raise ValueError("block_tables / q_starts / ctx_lens must be contiguous int32")
+    out = torch.empty((rows, heads * vdim), dtype=qkv.dtype, device=qkv.device)
+    if not decode:
+        splits = 1
+    elif splits <= 0:
+        ratio = heads // kv_heads
+        ctas = seqs * kv_heads * ((ratio + 3) // 4 if ratio > 2 else 1)
+        most = (window + 63) // 64 if window > 0 else 8
+        splits = max(1, min(8, most, 296 // max(1, ctas)))
+    ws = _zeroed_scratch("window_attention", qkv.device,
+                         lib().dz_window_attention_workspace_bytes(seqs, heads, kv_heads, vdim, splits))
+    args = _lib.WindowAttentionArgs(
+        qkv=qkv.data_ptr(), row_stride=qkv.stride(0), k_off=heads * dim, v_off=(heads + kv_heads) * dim,
+        out=out.data_ptr(), k_cache=k_cache.data_ptr(), v_cache=v_cache.data_ptr(),
+        block_tables=block_tables.data_ptr(), ring_blocks=block_tables.shape[1], block_size=block_size,
+        q_starts=q_starts.data_ptr(), ctx_lens=ctx_lens.data_ptr(), num_seqs=seqs, rows=rows, max_q=max_query,
+        decode=int(decode), heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=float(scale), window=window,
+        bias=_ptr(bias), bias_len=bias.shape[1] if bias is not None else 0, splits=splits,
+        workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=_any_dtype_code(qkv))
+    check(lib().dz_window_attention(ctypes.byref(args), _stream()), "dz_window_attention")
+    return out
+
+
+def mlstm_chunk_supported(dim: int, vdim: int, dtype: torch.dtype) -> bool:
+    code = {torch.float16: _lib.DZ_DTYPE_F16, torch.bfloat16: _lib.DZ_DTYPE_BF16}.get(dtype, _lib.DZ_DTYPE_F32)
+    return bool(lib().dz_mlstm_chunk_supported(dim, vdim, code))
+
+
+def mlstm(x: torch.Tensor, h: torch.Tensor, w_if: torch.Tensor, b_if: torch.Tensor, norm_weight: torch.Tensor,
+          S: torch.Tensor, n: torch.Tensor, m: torch.Tensor, slots: torch.Tensor, q_starts: torch.Tensor,
+          ctx_lens: torch.Tensor, gate_cap: float, scale: float, eps: float, chunkwise: bool) -> torch.Tensor:
+    """Matrix-memory recurrence, head norm and output gate over rows [q | k | v | g | ...]; the states
+    in slots `slots` are updated in place (dz_mlstm).  Returns [rows, heads * vdim]."""
+    _need_cuda(x, h, w_if, b_if, norm_weight, S, n, m, slots, q_starts, ctx_lens)
+    heads, dim, vdim = S.shape[1:]
+    rows, seqs = x.shape[0], ctx_lens.shape[0]
+    if any(t.dtype != torch.int32 or not t.is_contiguous() for t in (slots, q_starts, ctx_lens)):
+        raise ValueError("slots / q_starts / ctx_lens must be contiguous int32")
+    out = torch.empty((rows, heads * vdim), dtype=x.dtype, device=x.device)
+    pre = matmul_f32(h, w_if) if chunkwise else None
+    ws = _zeroed_scratch("mlstm", x.device, lib().dz_mlstm_workspace_bytes(seqs, heads)) if chunkwise else None
+    args = _lib.MlstmArgs(
+        x=x.data_ptr(), row_stride=x.stride(0), k_off=heads * dim, v_off=2 * heads * dim,
+        g_off=2 * heads * dim + heads * vdim, h=h.data_ptr(), w_if=w_if.data_ptr(), b_if=b_if.data_ptr(),
+        pre_if=_ptr(pre), width=h.shape[1], cap=float(gate_cap), scale=float(scale),
+        norm_weight=norm_weight.data_ptr(), eps=float(eps), out=out.data_ptr(), S=S.data_ptr(), n=n.data_ptr(),
+        m=m.data_ptr(), slots=slots.data_ptr(), q_starts=q_starts.data_ptr(), ctx_lens=ctx_lens.data_ptr(),
+        num_seqs=seqs, rows=rows, heads=heads, dim=dim, vdim=vdim, chunkwise=int(chunkwise),
+        workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=_any_dtype_code(x))
+    check(lib().dz_mlstm(ctypes.byref(args), _stream()), "dz_mlstm")
     return out

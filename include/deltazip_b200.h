@@ -37,7 +37,7 @@ typedef enum {
   DZ_ERR_TOO_LARGE = 11     /* size beyond a fixed maximum of the entry point   */
 } dz_status;
 
-enum { DZ_DTYPE_F16 = 0, DZ_DTYPE_BF16 = 1, DZ_DTYPE_F32 = 2 /* all-reduce only */ };
+enum { DZ_DTYPE_F16 = 0, DZ_DTYPE_BF16 = 1, DZ_DTYPE_F32 = 2 /* all-reduce and the 32-bit decoder steps */ };
 enum { DZ_INDEX_I32 = 0, DZ_INDEX_I64 = 1 };
 
 /* Library version (major*10000 + minor*100 + patch). */
@@ -303,6 +303,106 @@ int dz_sparsegpt_block(const float* W_block, int64_t ldw, const float* hinv_bloc
                        float* Err, float* loss, void* stream);
 int dz_pack_gptq(const float* Wq, const float* scale, const float* zero, int N, int K, int bits,
                  int32_t* qweight, int32_t* qzeros, uint16_t* scales, void* stream);
+
+/*
+ * Decoder steps with a 32-bit residual stream (any width; DZ_DTYPE_F16 / BF16 / F32 activations).
+ * A norm is x / sqrt(mean(x^2) + eps) * (weight_offset + weight), weights in 32 bits: offset 0 is the
+ * plain RMS norm, 1 the form whose weight is stored around zero.
+ *
+ *   embed_norm     residual = norm(table[token]); with `copy`, the same rounded to dtype goes to a
+ *                  column slice of a wider matrix (copy_stride elements per row)
+ *   residual_norm  residual = (replace ? 0 : residual) + delta + vec; out = norm(residual), or the
+ *                  residual itself when weight is NULL.  delta: dtype or DZ_DTYPE_F32; delta and vec
+ *                  may be NULL
+ *   gated_act      out[m, i] = act(x[m, i]) * x[m, inter + i]
+ */
+#define DZ_ACT_SILU 0
+#define DZ_ACT_GELU_TANH 1
+int dz_embed_norm(const int64_t* tokens, const void* table, int64_t vocab, const float* weight, float weight_offset,
+                  float* residual, void* copy, int64_t copy_stride, int M, int width, float eps, int dtype,
+                  void* stream);
+int dz_residual_norm(float* residual, const void* delta, int delta_dtype, int replace, const float* vec,
+                     const float* weight, float weight_offset, void* out, int64_t out_stride, int M, int width,
+                     float eps, int dtype, void* stream);
+int dz_gated_act(const void* x, int64_t x_stride, void* out, int M, int inter, int act, int dtype, void* stream);
+
+/*
+ * Sliding-window attention with a learned bias per distance over a ring of cache blocks
+ * (dz_window_attention.cu).  Rows are [q | k | v | ...]; row r of sequence s (q_starts[s] <= r <
+ * q_starts[s + 1]) has position ctx_lens[s] + r - q_starts[s].  score = (q.k) * scale +
+ * bias[head, min(distance, bias_len - 1)], visible for 0 <= distance < window (window <= 0: no
+ * lower bound).  Position t is cached in slot table[(t / block_size) % ring_blocks] * block_size +
+ * t % block_size.  decode = 0: keys at positions >= ctx_lens[s] come from the rows themselves and
+ * are appended with dz_kv_append afterwards; decode = 1 (one row per sequence): the row's key and
+ * value are in the cache already (dz_qk_norm with slot_mapping).  With splits > 1 the workspace must
+ * be zero-filled once before its first use.
+ */
+typedef struct dz_window_attention_args {
+  const void* qkv;
+  int64_t row_stride;
+  int32_t k_off, v_off;
+  void* out;
+  const void* k_cache;
+  const void* v_cache;
+  const int32_t* block_tables;
+  int32_t ring_blocks, block_size;
+  const int32_t* q_starts;
+  const int32_t* ctx_lens;
+  int32_t num_seqs, rows, max_q, decode;
+  int32_t heads, kv_heads, dim, vdim;
+  float scale;
+  int32_t window;
+  const float* bias;
+  int32_t bias_len, splits;
+  void* workspace;
+  size_t workspace_bytes;
+  int32_t dtype;
+} dz_window_attention_args;
+size_t dz_window_attention_workspace_bytes(int num_seqs, int heads, int kv_heads, int vdim, int splits);
+int dz_window_attention(const dz_window_attention_args* args, void* stream);
+/* RMS norm of the whole q row and of the whole k row in place (plain weights); with slot_mapping
+ * (one slot per row, < 0 = none) the normed k and v also go to the cache. */
+int dz_qk_norm(void* qkv, int64_t row_stride, int q_width, int k_width, int v_width, const float* wq, const float* wk,
+               float eps, void* k_cache, void* v_cache, const int64_t* slot_mapping, int M, int dtype, void* stream);
+int dz_kv_append(const void* qkv, int64_t row_stride, int k_off, int k_width, int v_width, void* k_cache,
+                 void* v_cache, const int64_t* slot_mapping, int M, int dtype, void* stream);
+
+/*
+ * Matrix-memory recurrence with exponential gates, its per-head output norm and output gate
+ * (dz_mlstm.cu).  Rows are [q | k | v | g] (heads * dim, heads * dim, heads * vdim, heads * vdim); the
+ * state pools S [slots, heads, dim, vdim], n [slots, heads, dim], m [slots, heads] are 32-bit and
+ * updated in place; a sequence with ctx_lens 0 starts from zero without reading its slot.
+ * chunkwise = 0: token after token, gates from h [rows, width] and w_if [2 heads, width] (w_i, w_f);
+ * chunkwise = 1 (dz_mlstm_chunk_supported): 64 tokens at a time, gates from pre_if [rows, 2 heads];
+ * the workspace must be zero-filled once before its first use.
+ */
+typedef struct dz_mlstm_args {
+  const void* x;
+  int64_t row_stride;
+  int32_t k_off, v_off, g_off;
+  const void* h;
+  const void* w_if;
+  const float* b_if;
+  const float* pre_if;
+  int32_t width;
+  float cap, scale;
+  const float* norm_weight;
+  float eps;
+  void* out;
+  float* S;
+  float* n;
+  float* m;
+  const int32_t* slots;
+  const int32_t* q_starts;
+  const int32_t* ctx_lens;
+  int32_t num_seqs, rows, heads, dim, vdim, chunkwise;
+  void* workspace;
+  size_t workspace_bytes;
+  int32_t dtype;
+} dz_mlstm_args;
+int dz_mlstm_chunk_supported(int dim, int vdim, int dtype);
+size_t dz_mlstm_workspace_bytes(int num_seqs, int heads);
+int dz_mlstm(const dz_mlstm_args* args, void* stream);
 
 /*
  * Delta swap-in: one asynchronous host->device copy of a delta's slot bytes
