@@ -838,7 +838,12 @@ sbmm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         c_first = split_owner(tile, 0, p.grid, KU, p.epi_units, U);
         nfrag = split_owner(tile, KU - 1, p.grid, KU, p.epi_units, U) - c_first + 1;
         slot_first = (split_begin(c_first, p.grid, KU, p.epi_units, U) / KU == tile) ? 0u : 1u;
-        if (ep_tid == 0) ticket = atomicAdd(&p.counters[2 * tile], 1);
+        if (ep_tid == 0) {
+          // a fragment without windows gets here before its x has arrived: in the early-start form
+          // the predecessor, perhaps another launch on the same counters, may still be running
+          if (p.stable) asm volatile("griddepcontrol.wait;" ::: "memory");
+          ticket = atomicAdd(&p.counters[2 * tile], 1);
+        }
       }
       // D_delta holds sums of (code - zero) * x; the per-channel scale of each
       // column's slot is applied here.  The scales are requested before the wait for the

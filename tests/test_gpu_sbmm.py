@@ -335,3 +335,20 @@ def test_prefill_runs_known_on_the_host_take_the_dequantise_once_path(bits):
     ids = [0] * 300 + [7] * 600 + [9] * 700
     _, (is_sorted, runs) = _convert_mapping(DeltaMapping(ids, [0, 7, 9]), [7, 9, None], 4, 32000, 0, device=dev)
     assert is_sorted and runs == [(-1, 0, 300), (0, 300, 900), (1, 900, 1600)]
+
+
+@pytest.mark.parametrize("m", [129, 151, 300, 512])
+@pytest.mark.parametrize("n,k", [(128, 512), (1280, 2048), (256, 128), (384, 192)])
+def test_early_start_launches_back_to_back_share_the_workspace(m, n, k):
+    """More than one token block per call and calls right behind one another, in the early-start form:
+    the launches settle their split tiles through the same counters and must not meet there."""
+    from deltazip_b200 import ops
+    g = torch.Generator(device="cuda").manual_seed(m + n)
+    x = torch.randn((m, k), generator=g, device="cuda").bfloat16()
+    w = torch.randn((n, k), generator=g, device="cuda").bfloat16()
+    want = x.float() @ w.float().t()
+    outs = [ops.base_gemm(x, w, stable=True) for _ in range(6)]
+    torch.cuda.synchronize()
+    for y in outs:
+        assert ((y.float() - want).norm() / want.norm()).item() < TOL
+    assert ops.read_status() == 0
