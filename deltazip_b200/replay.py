@@ -4,12 +4,12 @@
 
 Standard input holds one JSON object per line,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "left", "tokens": [11, 4], "want": [1]}], "end": ["left"]}
 
-`entries`: for each request its next tokens and the places among them whose logits are asked for;
-`end`: requests that are finished after the step.  A step that wants anything leaves
-DIR/<step>.f32, little-endian float32 [wanted, vocab] in the order of the entries and of `want`;
-every step is answered with a line "done <step>".  Nothing is sampled: the tokens go through
+with the next tokens of some requests, the indexes (within these tokens) whose logits are to be
+kept, and the requests that give back their cache and state once the step is through.  A step that
+keeps any leaves DIR/<step>.f32 (little-endian float32, one vocabulary row each, entry by entry);
+"done <step>" on standard output answers every step.  Nothing is sampled: the tokens go through
 DecodeEngine.extend, the forward pass that generation uses."""
 from __future__ import annotations
 

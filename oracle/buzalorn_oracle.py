@@ -65,6 +65,20 @@ def distance_bias(t, rel_column, bias_max):
     return np.where(i >= j, per[np.clip(i - j, 0, t - 1)], 0.0)
 
 
+def attention_core(q, k, v, scale, window, rel=None, bias_max=None):
+    """q [T, heads, dim], k [T, kv_heads, dim], v [T, kv_heads, vdim] -> [T, heads, vdim]."""
+    t, heads = q.shape[:2]
+    seen = window_visible(t, window)
+    out = np.empty((t, heads, v.shape[2]), dtype=q.dtype)
+    for a in range(heads):
+        g = a // (heads // k.shape[1])
+        s = q[:, a] @ k[:, g].T * scale
+        if rel is not None:
+            s = s + distance_bias(t, rel[:, a], bias_max)
+        out[:, a] = attention_weights(s, seen) @ v[:, g]
+    return out
+
+
 def attention(h, w, mix, eps):
     """w: dict with q, k, v, q.norm, k.norm, rel, o."""
     t = h.shape[0]
@@ -72,13 +86,8 @@ def attention(h, w, mix, eps):
     q = (rms_norm(h @ w["q"].T, eps) * w["q.norm"]).reshape(t, heads, dim)
     k = (rms_norm(h @ w["k"].T, eps) * w["k.norm"]).reshape(t, kvh, dim)
     v = (h @ w["v"].T).reshape(t, kvh, vdim)
-    seen = window_visible(t, mix["mask"]["size"])
-    out = np.empty((t, heads, vdim), dtype=h.dtype)
-    for a in range(heads):
-        g = a // (heads // kvh)
-        s = q[:, a] @ k[:, g].T * mix["scale"] + distance_bias(t, w["rel"][:, a], mix["bias_max"])
-        out[:, a] = attention_weights(s, seen) @ v[:, g]
-    return out.reshape(t, heads * vdim) @ w["o"].T
+    o = attention_core(q, k, v, mix["scale"], mix["mask"]["size"], w["rel"], mix["bias_max"])
+    return o.reshape(t, heads * vdim) @ w["o"].T
 
 
 def mlstm_recurrence(q, k, v, i, f):
@@ -98,18 +107,26 @@ def mlstm_recurrence(q, k, v, i, f):
     return out
 
 
+def mlstm_gates(pre_i, pre_f, cap):
+    """Log input and log forget gate from their pre-activations."""
+    return cap * np.tanh(pre_i / cap), log_sigmoid(cap * np.tanh(pre_f / cap))
+
+
+def head_norm_gate(o, norm, g, eps):
+    """o [T, heads, vdim] normed per head, times norm and sigmoid(g) -> [T, heads * vdim]."""
+    return rms_norm(o, eps).reshape(o.shape[0], -1) * norm * sigmoid(g)
+
+
 def mlstm(h, w, mix, eps):
     """w: dict with q, k, v, g, o, norm, i, i.b, f, f.b."""
     t = h.shape[0]
-    heads, dim, vdim, cap = mix["heads"], mix["dim"], mix["vdim"], mix["gate_cap"]
+    heads, dim, vdim = mix["heads"], mix["dim"], mix["vdim"]
     q = (h @ w["q"].T * dim ** -0.5).reshape(t, heads, dim)
     k = (h @ w["k"].T).reshape(t, heads, dim)
     v = (h @ w["v"].T).reshape(t, heads, vdim)
-    i = cap * np.tanh((h @ w["i"].T + w["i.b"]) / cap)
-    f = log_sigmoid(cap * np.tanh((h @ w["f"].T + w["f.b"]) / cap))
-    o = np.stack([rms_norm(mlstm_recurrence(q[:, a], k[:, a], v[:, a], i[:, a], f[:, a]), eps)
-                  for a in range(heads)], axis=1).reshape(t, heads * vdim)
-    return (o * w["norm"] * sigmoid(h @ w["g"].T)) @ w["o"].T
+    i, f = mlstm_gates(h @ w["i"].T + w["i.b"], h @ w["f"].T + w["f.b"], mix["gate_cap"])
+    o = np.stack([mlstm_recurrence(q[:, a], k[:, a], v[:, a], i[:, a], f[:, a]) for a in range(heads)], axis=1)
+    return head_norm_gate(o, w["norm"], h @ w["g"].T, eps) @ w["o"].T
 
 
 def layer_runs(config):
