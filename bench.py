@@ -17,6 +17,9 @@ request-to-delta map, tensor parallel.  --config 5: Llama-2-70B, 16 4-bit deltas
 memory, 4 GPU slots, bursty arrivals, swap-in overlapped with decode (--duration seconds of
 arrivals on a virtual clock).
 
+--arch buzalorn: prefill and decode throughput of the Buzalorn decoder beside the Llama decoder at
+equal sizes, and the kernels of both against their rooflines (deltazip_b200/model_bench.py).
+
 N > 1: tensor parallel over N ranks (column-parallel qkv / gate_up, row-parallel o / down
 followed by the library's peer-memory all-reduce), shards cut at whole 128-wide units; the total
 work is fixed ("strong" scaling).
@@ -544,9 +547,11 @@ def measured_peaks():
     path = os.path.join(ROOT, "MEASURED_PEAKS.json")
     try:
         with open(path) as fh:
-            return {"hbm_gbs": float(json.load(fh)["hbm_gbs"]), "source": "measured (MEASURED_PEAKS.json)"}
+            d = json.load(fh)
+            return {"hbm_gbs": float(d["hbm_gbs"]), "bf16_tflops": float(d.get("bf16_tflops", 1590.0)),
+                    "source": "measured (MEASURED_PEAKS.json)"}
     except (OSError, KeyError, ValueError):
-        return {"hbm_gbs": 6650.0, "source": "fallback (6.65 TB/s)"}
+        return {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback (6.65 TB/s, 1.59 PFLOP/s)"}
 
 
 def ncu_traffic_per_launch(alg_bytes_per_launch):
@@ -1277,7 +1282,15 @@ def main():
                     help="config 5: seconds of simulated arrivals (default 300)")
     ap.add_argument("--wall-limit", type=float, default=None,
                     help="config 5: stop the serving loop after this many wall-clock seconds (default 600)")
+    ap.add_argument("--arch", default=None, choices=["buzalorn"],
+                    help="instead of a configuration: this decoder beside the Llama decoder at equal sizes, whole "
+                         "models and kernel by kernel")
+    ap.add_argument("--size", default=None, help="--arch: only these sizes (comma-separated)")
     args = ap.parse_args()
+    if args.arch:
+        from deltazip_b200 import model_bench
+        print(json.dumps(model_bench.run(args, measured_peaks(), ClockSampler(0))), flush=True)
+        return
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
     if args.config in DECODE_CONFIGS:
