@@ -15,33 +15,10 @@
 //
 // Scores, softmax weights and sums are 32-bit.  In the tensor-core kernel a weight enters its
 // product with v as a hi + lo pair of 16-bit numbers.
-#include "dz_elem.cuh"
+#include "dz_window_attention.cuh"
 
 namespace dz {
 namespace {
-
-struct AttnParams {
-  const void* qkv;
-  int64_t row_stride;                    // elements
-  int k_off, v_off;                      // columns where the key / value parts start
-  void* out;                             // [rows, heads * vdim]
-  const void* k_cache;                   // [slots, kv_heads, dim]
-  const void* v_cache;                   // [slots, kv_heads, vdim]
-  const int* block_tables;               // [sequences, ring_blocks]
-  int ring_blocks, block_size;
-  const int* q_starts;                   // [sequences + 1] first row of every sequence
-  const int* ctx_lens;                   // [sequences] tokens already in the cache
-  int heads, kv_heads, dim, vdim;
-  float scale;
-  int window;
-  const float* bias;                     // [heads, bias_len] or nullptr
-  int bias_len;
-};
-
-__device__ __forceinline__ size_t ring_slot(const AttnParams& p, const int* table, int t) {
-  const int b = t / p.block_size;
-  return (size_t)table[b % p.ring_blocks] * p.block_size + (t - b * p.block_size);
-}
 
 // -------------------------------------------------------------------------------------------------
 // RMS norm of the whole query row and of the whole key row (all heads at once), in place, and the
@@ -412,12 +389,12 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
 }
 
 // -------------------------------------------------------------------------------------------------
-// Prompt portions on the tensor cores: 64 query rows of one (sequence, head) per CTA, 16 per warp,
+// Short prompt portions, and sizes the tcgen05 kernel (dz_window_attention_tc.cu) does not take, on
+// warp-level MMAs: 64 query rows of one (sequence, head) per CTA, 16 per warp,
 // 64 keys per step, double-buffered through cp.async.  Grid (row tiles, heads x tiles of DVP value
 // columns, sequences).
 // -------------------------------------------------------------------------------------------------
 constexpr int kBM = 64, kBN = 64, kBiasSmem = 4096;
-constexpr float kLog2e = 1.4426950408889634f;
 
 template <typename T, int DVP>
 __global__ void __launch_bounds__(128)
@@ -638,6 +615,9 @@ int run_decode_g(const AttnParams& p, dim3 grid, int splits, float* partial, int
   return DZ_OK;
 }
 
+constexpr int kTcMinRows = 64;                 // portions up to this many rows stay off the 256-row kernel
+constexpr size_t kAttnStatusBytes = 256;        // workspace: [status word | tickets | partials]
+
 int decode_group(int heads, int kv_heads) {
   const int r = heads / kv_heads;
   return r == 1 ? 1 : r == 2 ? 2 : 4;
@@ -692,8 +672,9 @@ int dz_kv_append(const void* qkv, int64_t row_stride, int k_off, int k_width, in
 }
 
 size_t dz_window_attention_workspace_bytes(int num_seqs, int heads, int kv_heads, int vdim, int splits) {
-  if (num_seqs <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || vdim <= 0 || splits <= 1) return 0;
-  return ticket_bytes(num_seqs, heads, kv_heads) + (size_t)num_seqs * heads * splits * (vdim + 2) * 4;
+  if (num_seqs <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || vdim <= 0) return 0;
+  if (splits <= 1) return kAttnStatusBytes;
+  return kAttnStatusBytes + ticket_bytes(num_seqs, heads, kv_heads) + (size_t)num_seqs * heads * splits * (vdim + 2) * 4;
 }
 
 int dz_window_attention(const dz_window_attention_args* a, void* stream) {
@@ -711,7 +692,8 @@ int dz_window_attention(const dz_window_attention_args* a, void* stream) {
   if (a->num_seqs > 65535 || (a->decode && a->rows != a->num_seqs)) return DZ_ERR_INVALID_ARG;
   AttnParams p = {a->qkv, a->row_stride, a->k_off, a->v_off, a->out, a->k_cache, a->v_cache, a->block_tables,
                   a->ring_blocks, a->block_size, a->q_starts, a->ctx_lens, a->heads, a->kv_heads, a->dim, a->vdim,
-                  a->scale, a->window, a->bias, a->bias_len};
+                  a->scale, a->window, a->bias, a->bias_len, nullptr};
+  if (a->workspace && a->workspace_bytes >= kAttnStatusBytes) p.status = (int*)a->workspace;
   cudaStream_t st = (cudaStream_t)stream;
   if (!fast_shapes(p, a->dtype)) {
     if (a->vdim > kAnyMaxV * kAnyThreads || a->dim > 8192 || a->heads > 65535) return DZ_ERR_SHAPE;
@@ -726,8 +708,8 @@ int dz_window_attention(const dz_window_attention_args* a, void* stream) {
       if (!a->workspace || a->workspace_bytes < dz_window_attention_workspace_bytes(a->num_seqs, a->heads, a->kv_heads,
                                                                                     a->vdim, a->splits))
         return DZ_ERR_WORKSPACE;
-      tickets = (int*)a->workspace;
-      partial = (float*)((uint8_t*)a->workspace + ticket_bytes(a->num_seqs, a->heads, a->kv_heads));
+      tickets = (int*)((uint8_t*)a->workspace + kAttnStatusBytes);
+      partial = (float*)((uint8_t*)tickets + ticket_bytes(a->num_seqs, a->heads, a->kv_heads));
     }
     const dim3 grid(decode_grid_x(a->heads, a->kv_heads), a->num_seqs, a->splits);
     const int g = decode_group(a->heads, a->kv_heads);
@@ -735,11 +717,13 @@ int dz_window_attention(const dz_window_attention_args* a, void* stream) {
                                    : g == 2 ? run_decode_g<T, 2>(p, grid, a->splits, partial, tickets, st)
                                             : run_decode_g<T, 4>(p, grid, a->splits, partial, tickets, st));
   }
+  const int max_q = a->max_q > 0 ? a->max_q : a->rows;
+  if (max_q > kTcMinRows && window_prefill_tc_supported(p, a->dtype))
+    return launch_window_prefill_tc(p, a->num_seqs, max_q, a->dtype, st);
   const int dimp = (a->dim + 15) / 16 * 16;
   const int dvp = a->vdim <= 64 ? 64 : a->vdim <= 96 ? 96 : a->vdim <= 128 ? 128 : a->vdim <= 192 ? 192 : 256;
   const size_t bias_bytes = a->bias && a->bias_len <= kBiasSmem ? (size_t)a->bias_len * 4 : 0;
   const size_t smem = ((size_t)(kBM + 2 * kBN) * (dimp + 8) + (size_t)2 * kBN * (dvp + 8)) * 2 + bias_bytes;
-  const int max_q = a->max_q > 0 ? a->max_q : a->rows;
   if (smem > kMaxDynSmem || (int64_t)a->heads * ((a->vdim + dvp - 1) / dvp) > 65535) {
     if (a->vdim > kAnyMaxV * kAnyThreads || a->dim > 8192 || a->heads > 65535) return DZ_ERR_SHAPE;
     DZ_DISPATCH16(a->dtype, DZ_CUDA_OK(launch_ex(attention_any_kernel<T>, dim3(a->rows, a->heads), dim3(kAnyThreads),

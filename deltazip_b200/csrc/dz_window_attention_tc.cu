@@ -1,0 +1,373 @@
+// Sliding-window attention for prompt portions on the 5th-generation tensor cores.
+//
+// A CTA takes 256 query rows of one (sequence, head) as two tiles of 128 (the MMA's M, one row per
+// TMEM lane) and walks the keys in tiles of 128 that both read.  Roles of its twelve warps:
+//   0-3, 4-7  softmax of query tile 0 / 1: a thread owns a row -- scores from TMEM into registers,
+//             scale + bias + mask, running maximum, exponentials, weights back to TMEM
+//   8-9       copies: keys and values from the projection rows or the cache ring into 128-byte-swizzled
+//             shared memory, two stages
+//   10, 11    MMA issue for query tile 0 / 1: S = Q K^T (both operands in shared memory), O += P V
+//             (P in TMEM, V read as it lies, keys along K and value columns contiguous)
+// The two query tiles are independent chains, so one's softmax runs under the other's MMAs.
+//
+// TMEM: S0 | S1 | O0 | O1, 128 columns each.  The weights take the place of the scores they came from:
+// 64 columns of 16-bit pairs (hi) and 64 with what the rounding left (lo); two products with v keep
+// the weights at about 32-bit accuracy.
+//
+// The running maximum is only moved when it has grown by more than 8 (log2 units): weights then stay
+// below 2^8, sums stay exact, and most tiles need no pass over O.
+#include <algorithm>
+#include <type_traits>
+
+#include "dz_tc.cuh"
+#include "dz_window_attention.cuh"
+
+namespace dz {
+namespace {
+
+constexpr int kTileM = 128, kTileKeys = 128, kStages = 2;
+constexpr int kThreadsTc = 384, kCopyThreads = 64;
+constexpr int kSlab = 128 * 128;                        // 128 rows of 64 16-bit elements
+constexpr int kBiasTc = 4096;
+constexpr int kBiasPad = 254;                           // distances from -254 up are in the table
+constexpr float kMaxGrowth = 8.f;
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// byte offset of 16-byte chunk c of row r in a run of 64-element slabs
+__device__ __forceinline__ uint32_t swizzled(int r, int c) {
+  return (uint32_t)((c >> 3) * kSlab + r * 128 + (((c & 7) ^ (r & 7)) << 4));
+}
+
+__device__ __forceinline__ void cp_async16_u32(uint32_t dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+
+__device__ __forceinline__ void umma_ss(uint32_t d, uint32_t a_lo, uint32_t b_lo, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t.reg .b64 da, db;\n\t"
+      "setp.ne.b32 p, %5, 0;\n\t"
+      "mov.b64 da, {%1, %3};\n\tmov.b64 db, {%2, %3};\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %4, p;\n\t}" ::"r"(d),
+      "r"(a_lo), "r"(b_lo), "r"(kDescHi), "r"(idesc), "r"(acc)
+      : "memory");
+}
+__device__ __forceinline__ void umma_ts(uint32_t d, uint32_t a, uint32_t b_lo, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t.reg .b64 db;\n\t"
+      "setp.ne.b32 p, %5, 0;\n\t"
+      "mov.b64 db, {%2, %3};\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], db, %4, p;\n\t}" ::"r"(d),
+      "r"(a), "r"(b_lo), "r"(kDescHi), "r"(idesc), "r"(acc)
+      : "memory");
+}
+// v lies [key][column]: "MN-major", 64 columns (128 bytes) per slab, slabs one leading offset apart,
+// groups of eight keys 1024 bytes apart
+__device__ __forceinline__ uint32_t desc_lo_mn(uint32_t saddr) {
+  return ((saddr >> 4) & 0x3FFFu) | ((uint32_t)(kSlab >> 4) << 16);
+}
+
+__device__ __forceinline__ void tmem_ld32(uint32_t a, float* f) {
+  uint32_t* v = reinterpret_cast<uint32_t*>(f);
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
+      "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
+        "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
+        "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
+        "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+      : "r"(a)
+      : "memory");
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreadsTc, 1)
+window_prefill_tc_kernel(const AttnParams p) {
+  constexpr int DT = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
+  extern __shared__ uint8_t smem_dyn[];
+  __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2], b_p[2], b_o[2];
+  __shared__ uint32_t s_tmem;
+  __shared__ int s_abort;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int seq = blockIdx.z, head = blockIdx.y % p.heads, v0 = (blockIdx.y / p.heads) * 128;
+  pdl_wait();
+  pdl_launch();
+  const int q0 = p.q_starts[seq], qn = p.q_starts[seq + 1] - q0, ctx = p.ctx_lens[seq];
+  const int m0 = blockIdx.x * 2 * kTileM;
+  if (m0 >= qn) return;
+  const int kvh = head / (p.heads / p.kv_heads);
+  const int vcols = min(128, p.vdim - v0);
+  const int ks = (p.dim + 63) / 64, vs = (vcols + 63) / 64;      // slabs
+  const uint32_t s_base = (smem_u32(smem_dyn) + 1023u) & ~1023u;
+  const uint32_t s_q = s_base, s_k = s_q + 2 * ks * kSlab, s_v = s_k + kStages * ks * kSlab;
+  float* s_bias = reinterpret_cast<float*>(smem_dyn + (s_v + kStages * vs * kSlab - smem_u32(smem_dyn)));
+  volatile int* abort_flag = &s_abort;
+  const T* qkv = (const T*)p.qkv;
+  const int* table = p.block_tables + (size_t)seq * p.ring_blocks;
+
+  // key tiles: all of the CTA's, and of those the range [ta, tb) with keys a query tile may see
+  const int first = p.window > 0 ? max(0, ctx + m0 - p.window + 1) : 0;
+  const int end = ctx + min(m0 + 2 * kTileM, qn);
+  const int tiles = (end - first + kTileKeys - 1) / kTileKeys;
+  const int g = warp < 8 ? warp >> 2 : warp - 10;                // query tile of this warp (copy warps: unused)
+  const int w0 = ctx + m0 + g * kTileM;                          // position of the tile's first row
+  const int rows = min(kTileM, qn - m0 - g * kTileM);
+  const int lo = p.window > 0 ? max(0, w0 - p.window + 1) : 0;
+  const int ta = rows > 0 ? (lo - first) / kTileKeys : 0;
+  const int tb = rows > 0 ? (w0 + rows - first + kTileKeys - 1) / kTileKeys : 0;
+
+  if (tid == 0) {
+    for (int i = 0; i < kStages; ++i) {
+      mbar_init(smem_u32(&b_full[i]), kCopyThreads);
+      mbar_init(smem_u32(&b_empty[i]), 2);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(smem_u32(&b_s[i]), 1);
+      mbar_init(smem_u32(&b_p[i]), kTileM);
+      mbar_init(smem_u32(&b_o[i]), 1);
+    }
+    s_abort = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    fence_proxy_async();
+  }
+  if (warp == 10) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "n"(512)
+                 : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  if (p.dim % 16) {                                              // columns up to the MMA's K read as zero
+    for (uint32_t i = tid * 16; i < (uint32_t)(2 + kStages) * ks * kSlab; i += kThreadsTc * 16)
+      sts128(s_q + i, make_uint4(0, 0, 0, 0));
+    __syncthreads();
+  }
+  const int blen = p.bias ? p.bias_len : 1;
+  for (int i = tid; i < blen + 2 * kBiasPad; i += kThreadsTc) {
+    const int d = i - kBiasPad;
+    s_bias[i] = d < 0 ? -INFINITY : p.bias ? p.bias[(size_t)head * p.bias_len + min(d, blen - 1)] * kLog2e : 0.f;
+  }
+  if (warp < 8) {
+    const int c = tid & 15;
+    if (c < p.dim / 8) {
+      for (int r = tid >> 4; r < 2 * kTileM; r += 16) {
+        const bool ok = m0 + r < qn;
+        const T* src = qkv + (size_t)(q0 + (ok ? m0 + r : 0)) * p.row_stride + (size_t)head * p.dim + c * 8;
+        cp_async16_u32(s_q + (r >> 7) * ks * kSlab + swizzled(r & 127, c), src, ok);
+      }
+    }
+    cp_async_commit();
+    cp_async_wait<0>();
+  }
+  fence_proxy_async();                                           // queries and zeroed columns, for the MMAs
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = s_tmem;
+
+  if (warp >= 10) {
+    // ---- MMA issue ----
+    if (lane == 0) {
+      const uint32_t id_s = make_idesc<DT>(kTileKeys, false);
+      const uint32_t id_o = make_idesc<DT>(vs * 64, false) | (1u << 16);       // B transposed
+      const uint32_t t_s = tmem + g * 128, t_o = tmem + 256 + g * 128;
+      const int ksteps = (p.dim + 15) / 16;
+      auto scores = [&](int j) {
+        const int st = j & 1;
+        mbar_wait(smem_u32(&b_full[st]), (j >> 1) & 1, abort_flag, p.status);
+        tc_fence_after();
+        const uint32_t a = desc_lo(s_q + g * ks * kSlab), b = desc_lo(s_k + st * ks * kSlab);
+        for (int k = 0; k < ksteps; ++k) {
+          const uint32_t off = (uint32_t)((k >> 2) * (kSlab >> 4) + (k & 3) * 2);
+          umma_ss(t_s, a + off, b + off, id_s, k > 0);
+        }
+        umma_commit(smem_u32(&b_s[g]));
+      };
+      for (int j = 0; j < tiles; ++j) {
+        const int st = j & 1;
+        if (j < ta || j >= tb) {
+          mbar_wait(smem_u32(&b_full[st]), (j >> 1) & 1, abort_flag, p.status);
+          mbar_arrive(smem_u32(&b_empty[st]));
+          continue;
+        }
+        if (j == ta) scores(j);
+        mbar_wait(smem_u32(&b_p[g]), (j - ta) & 1, abort_flag, p.status);
+        tc_fence_after();
+        const uint32_t b = desc_lo_mn(s_v + st * vs * kSlab);
+#pragma unroll
+        for (int k = 0; k < kTileKeys / 16; ++k) {                              // 16 keys: 2048 bytes of v
+          umma_ts(t_o, t_s + k * 8, b + k * 128, id_o, (j > ta || k > 0) ? 1u : 0u);
+          umma_ts(t_o, t_s + 64 + k * 8, b + k * 128, id_o, 1u);
+        }
+        umma_commit(smem_u32(&b_empty[st]));
+        if (j + 1 < tb) scores(j + 1);             // behind the product that reads these columns' weights
+        else umma_commit(smem_u32(&b_o[g]));
+      }
+    }
+  } else if (warp >= 8) {
+    // ---- copies ----
+    const int t = tid - 256, c = t & 15;
+    for (int j = 0; j < tiles; ++j) {
+      const int st = j & 1;
+      mbar_wait(smem_u32(&b_empty[st]), ((j >> 1) & 1) ^ 1, abort_flag, p.status);
+      const uint32_t dk = s_k + st * ks * kSlab, dv = s_v + st * vs * kSlab;
+#pragma unroll 4
+      for (int r = t >> 4; r < kTileKeys; r += kCopyThreads / 16) {
+        const int key = first + j * kTileKeys + r;
+        const bool ok = key < end;
+        const T *kp, *vp;
+        if (!ok || key >= ctx) {
+          const T* row = qkv + (size_t)(q0 + (ok ? key - ctx : 0)) * p.row_stride;
+          kp = row + p.k_off + (size_t)kvh * p.dim;
+          vp = row + p.v_off + (size_t)kvh * p.vdim;
+        } else {
+          const size_t slot = ring_slot(p, table, key) * p.kv_heads + kvh;
+          kp = (const T*)p.k_cache + slot * p.dim;
+          vp = (const T*)p.v_cache + slot * p.vdim;
+        }
+        const uint32_t at = swizzled(r, c);
+        if (c < p.dim / 8) cp_async16_u32(dk + at, kp + c * 8, ok);
+        if (c < vcols / 8) cp_async16_u32(dv + at, vp + v0 + c * 8, ok);
+      }
+      cp_async_commit();
+      cp_async_wait<0>();
+      fence_proxy_async();
+      mbar_arrive(smem_u32(&b_full[st]));
+    }
+  } else if (rows > 0) {
+    // ---- softmax ----
+    const int r = (warp & 3) * 32 + lane, pos = w0 + r;
+    const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+    const uint32_t t_s = tmem + g * 128 + lane_addr, t_o = tmem + 256 + g * 128 + lane_addr;
+    const float scale2 = p.scale * kLog2e, far_bias = s_bias[kBiasPad + blen - 1];
+    float m = -INFINITY, l = 0.f;
+    for (int j = ta; j < tb; ++j) {
+      mbar_wait(smem_u32(&b_s[g]), (j - ta) & 1, abort_flag, p.status);
+      tc_fence_after();
+      float s[kTileKeys];
+#pragma unroll
+      for (int c = 0; c < kTileKeys; c += 32) tmem_ld32(t_s + c, s + c);
+      tmem_wait_ld();
+      const int t0 = first + j * kTileKeys;
+      if (w0 - (t0 + kTileKeys - 1) >= blen - 1) {               // every distance is in the last column
+#pragma unroll
+        for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, far_bias);
+      } else {                                                    // minus infinity at negative distances
+        const float* tb_ = s_bias + kBiasPad + (pos - t0);
+#pragma unroll
+        for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, tb_[-c]);
+      }
+      if (p.window > 0 && w0 + kTileM - 1 - t0 >= p.window) {
+        const int out = pos - p.window - t0;                      // keys up to here have left the window
+#pragma unroll
+        for (int c = 0; c < kTileKeys; ++c) s[c] = c <= out ? -INFINITY : s[c];
+      }
+      float mx[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+      for (int c = 4; c < kTileKeys; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
+      const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+      float f = 1.f;
+      if (m == -INFINITY) {
+        m = top;                                                  // nothing summed so far
+      } else if (top > m + kMaxGrowth) {
+        f = ex2(m - top);
+        m = top;
+        l *= f;
+      }
+      const bool rescale = __any_sync(0xffffffffu, f != 1.f);
+      const float ms = m == -INFINITY ? 0.f : m;
+      float sum[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int c = 0; c < kTileKeys; c += 32) {
+        uint32_t hi[16], low[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float a = ex2(s[c + 2 * i] - ms), b = ex2(s[c + 2 * i + 1] - ms);
+          sum[(2 * i) & 3] += a;
+          sum[(2 * i + 1) & 3] += b;
+          split_pair<T>(a, b, hi[i], low[i]);
+        }
+        tmem_st16(t_s + c / 2, hi);
+        tmem_st16(t_s + 64 + c / 2, low);
+      }
+      l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
+      if (rescale) {                                              // the product before is complete: its commit is b_s
+        for (int c = 0; c < vs * 64; c += 32) {
+          float o[32];
+          tmem_ld32(t_o + c, o);
+          tmem_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) o[i] *= f;
+          tmem_st16(t_o + c, reinterpret_cast<const uint32_t*>(o));
+          tmem_st16(t_o + c + 16, reinterpret_cast<const uint32_t*>(o + 16));
+        }
+      }
+      tmem_wait_st();
+      tc_fence_before();
+      mbar_arrive(smem_u32(&b_p[g]));
+    }
+    mbar_wait(smem_u32(&b_o[g]), 0, abort_flag, p.status);
+    tc_fence_after();
+    const float inv = 1.f / l;
+    T* op = (T*)p.out + (size_t)(q0 + m0 + g * kTileM + r) * p.heads * p.vdim + (size_t)head * p.vdim + v0;
+    for (int c = 0; c < vcols; c += 32) {
+      float o[32];
+      tmem_ld32(t_o + c, o);
+      tmem_wait_ld();
+      if (r < rows) {
+#pragma unroll
+        for (int i = 0; i < 32; i += 8) {
+          if (c + i < vcols) {
+            float v[8];
+#pragma unroll
+            for (int q = 0; q < 8; ++q) v[q] = o[i + q] * inv;
+            store8<T>(op + c + i, v);
+          }
+        }
+      }
+    }
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (s_abort) {                                                  // let issued MMAs end before TMEM goes
+    const unsigned long long t0 = globaltimer();
+    while (globaltimer() - t0 < 200000ull) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (warp == 10) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(512) : "memory");
+  }
+}
+
+size_t tc_smem(const AttnParams& p) {
+  const int ks = (p.dim + 63) / 64, vs = (std::min(128, p.vdim) + 63) / 64;
+  const int blen = p.bias ? p.bias_len : 1;
+  return (size_t)((2 + kStages) * ks + kStages * vs) * kSlab + (size_t)(blen + 2 * kBiasPad) * 4 + 1024;
+}
+
+template <typename T>
+int run(const AttnParams& p, int num_seqs, int max_q, cudaStream_t st) {
+  const size_t smem = tc_smem(p);
+  const dim3 grid((max_q + 2 * kTileM - 1) / (2 * kTileM), p.heads * ((p.vdim + 127) / 128), num_seqs);
+  DZ_CUDA_OK(allow_smem(window_prefill_tc_kernel<T>, smem));
+  DZ_CUDA_OK(launch_ex(window_prefill_tc_kernel<T>, grid, dim3(kThreadsTc), smem, 1, st, p));
+  return DZ_OK;
+}
+
+}  // namespace
+
+bool window_prefill_tc_supported(const AttnParams& p, int dtype) {
+  return (dtype == DZ_DTYPE_F16 || dtype == DZ_DTYPE_BF16) && p.dim <= 128 && p.dim % 8 == 0 && p.vdim % 8 == 0 &&
+         (!p.bias || p.bias_len <= kBiasTc) && p.heads * ((p.vdim + 127) / 128) <= 65535;
+}
+
+int launch_window_prefill_tc(const AttnParams& p, int num_seqs, int max_q, int dtype, cudaStream_t st) {
+  return dtype == DZ_DTYPE_BF16 ? run<__nv_bfloat16>(p, num_seqs, max_q, st) : run<__half>(p, num_seqs, max_q, st);
+}
+
+}  // namespace dz

@@ -175,16 +175,18 @@ def _workspace(device, nbytes: int) -> torch.Tensor:
 
 
 def read_status(device=None) -> int:
-    """Reads and clears the status word the SBMM kernel leaves in the current
-    stream's workspace (0 = ok, DZ_ERR_TIMEOUT = a bounded device-side wait ran
+    """Reads and clears the status words the SBMM and the window attention kernels leave in the
+    current stream's workspaces (0 = ok, DZ_ERR_TIMEOUT = a bounded device-side wait ran
     out, DZ_ERR_INVALID_ARG = a wrong `tokens_sorted` promise).  Synchronises."""
     device = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
-    ws = _workspaces.get((device.index, _stream()))
-    if ws is None:
-        return 0
-    host = ctypes.c_int(0)
-    check(lib().dz_read_status(ws.data_ptr(), _stream(), ctypes.byref(host)), "dz_read_status")
-    return host.value
+    found = 0
+    for ws in (_workspaces.get((device.index, _stream())),
+               _scratch.get(("window_attention", device.index, _stream()))):
+        if ws is not None:
+            host = ctypes.c_int(0)
+            check(lib().dz_read_status(ws.data_ptr(), _stream(), ctypes.byref(host)), "dz_read_status")
+            found = found or host.value
+    return found
 
 
 def _dtype_code(t: torch.Tensor) -> int:

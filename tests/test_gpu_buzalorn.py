@@ -117,7 +117,7 @@ class AttentionRun:
         cut = np.split(host(self.rows), np.cumsum(self.parts)[:2], axis=1)
         self.want = O.attention_core(cut[0].reshape(q.shape), cut[1].reshape(k.shape), cut[2].reshape(v.shape),
                                      scale, window, rel_table, bias_max)
-        self.cache = PagedKVCache(1, 40, kvh, block, dtype, "cuda", layer_shapes=[(kvh, dim, vdim)], window=window)
+        self.cache = PagedKVCache(1, 70, kvh, block, dtype, "cuda", layer_shapes=[(kvh, dim, vdim)], window=window)
         self.cache.k[0].fill_(float("nan"))             # nothing may be read that was not written
         self.cache.v[0].fill_(float("nan"))
         self.cache.allocate(spare)
@@ -163,6 +163,24 @@ def test_attention_kernels(shape, dtype):
         for splits in (0, 3):
             assert rel(r.run(cuts, splits), r.want) < EXACT[dtype], (cuts, splits)
     assert rel(r.run([70, 1, 1, 30], decode_single=False), r.want) < EXACT[dtype]
+
+
+@pytest.mark.parametrize("shape", [(2, 1, 128, 128), (2, 2, 64, 64), (3, 1, 72, 104), (1, 1, 40, 200)])
+@pytest.mark.parametrize("window", [129, 300, 5000])
+@pytest.mark.parametrize("dtype", [F16, BF16])
+def test_attention_long_portions(shape, window, dtype):
+    """Several 256-row blocks of the tcgen05 kernel, with and without context, running maxima that grow
+    along the keys, and a table longer than a key tile."""
+    heads, kvh, dim, vdim = shape
+    rng = np.random.default_rng(window + dim)
+    t = 900
+    q, k, v = (rng.normal(size=(t, n, d)) for n, d in ((heads, dim), (kvh, dim), (kvh, vdim)))
+    k *= np.linspace(0.2, 3.0, t)[:, None, None]
+    r = AttentionRun(q, k, v, dtype, window, 1.5 * dim ** -0.5, rng.normal(size=(32, heads)) * 2, 200, block=16)
+    for cuts in ([t], [257, 643], [100, 65, 300, 128, 307]):
+        assert rel(r.run(cuts), r.want) < EXACT[dtype], cuts
+    from deltazip_b200 import ops
+    assert ops.read_status() == 0
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
