@@ -692,7 +692,7 @@ int dz_window_attention(const dz_window_attention_args* a, void* stream) {
   if (a->num_seqs > 65535 || (a->decode && a->rows != a->num_seqs)) return DZ_ERR_INVALID_ARG;
   AttnParams p = {a->qkv, a->row_stride, a->k_off, a->v_off, a->out, a->k_cache, a->v_cache, a->block_tables,
                   a->ring_blocks, a->block_size, a->q_starts, a->ctx_lens, a->heads, a->kv_heads, a->dim, a->vdim,
-                  a->scale, a->window, a->bias, a->bias_len, nullptr};
+                  a->scale, a->window, a->bias, a->bias_len, a->rows, nullptr};
   if (a->workspace && a->workspace_bytes >= kAttnStatusBytes) p.status = (int*)a->workspace;
   cudaStream_t st = (cudaStream_t)stream;
   if (!fast_shapes(p, a->dtype)) {

@@ -21,6 +21,7 @@ struct AttnParams {
   int window;
   const float* bias;                     // [heads, bias_len] or nullptr
   int bias_len;
+  int rows;                              // of qkv
   int* status;                           // first error a kernel met (sticky until read)
 };
 

