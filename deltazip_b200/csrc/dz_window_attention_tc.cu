@@ -98,12 +98,20 @@ __device__ __forceinline__ void tmem_ld32(uint32_t a, float* f) {
       : "memory");
 }
 
+// Bounded wait that polls (each try suspends for a while by itself) before it falls back to sleeping.
+__device__ __forceinline__ void bar_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int* status) {
+#pragma unroll 1
+  for (int i = 0; i < 32; ++i)
+    if (mbar_try_wait(smem_u32(bar), parity)) return;
+  mbar_wait_slow(smem_u32(bar), parity, abort_flag, status);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kThreadsTc, 1)
 window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnParams p) {
   constexpr int DT = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
   extern __shared__ uint8_t smem_dyn[];
-  __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2][2], b_p[2][2], b_pv[2], b_o[2];
+  __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2][2], b_p[2][2], b_pv[2], b_o[2], b_q;
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -142,11 +150,12 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
     for (int i = 0; i < 2; ++i) {
       for (int k = 0; k < 2; ++k) {
         mbar_init(smem_u32(&b_s[i][k]), 1);
-        mbar_init(smem_u32(&b_p[i][k]), kTileM);
+        mbar_init(smem_u32(&b_p[i][k]), kTileM / 32);
       }
       mbar_init(smem_u32(&b_pv[i]), 1);
       mbar_init(smem_u32(&b_o[i]), 1);
     }
+    mbar_init(smem_u32(&b_q), 9);                                // eight softmax warps, one copy thread
     s_abort = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     fence_proxy_async();
@@ -162,26 +171,12 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
     __syncthreads();
   }
   const int blen = p.bias ? p.bias_len : 1;
-  for (int i = tid; i < blen + 2 * kBiasPad; i += kThreadsTc) {
-    const int d = i - kBiasPad;
-    s_bias[i] = d < 0 ? -INFINITY : p.bias ? p.bias[(size_t)head * p.bias_len + min(d, blen - 1)] * kLog2e : 0.f;
-  }
-  if (warp < 8) {
-    const int c = tid & 15;
-    if (c < p.dim / 8) {
-      for (int r = tid >> 4; r < 2 * kTileM; r += 16) {
-        const bool ok = m0 + r < qn;
-        const T* src = qkv + (size_t)(q0 + (ok ? m0 + r : 0)) * p.row_stride + (size_t)head * p.dim + c * 8;
-        cp_async16_u32(s_q + (r >> 7) * ks * kSlabQ + swizzled(r & 127, c, kSlabQ), src, ok);
-      }
-    }
-    cp_async_commit();
-    cp_async_wait<0>();
-  }
-  fence_proxy_async();                                           // queries and zeroed columns, for the MMAs
+  fence_proxy_async();                                           // zeroed columns, for the MMAs
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  // queries come by TMA where the 256 rows and their columns are all the sequence's and head's own
+  const bool q_tma = p.dim % 16 == 0 && m0 + 2 * kTileM <= qn;
   const uint32_t tmem = s_tmem;
 
   if (warp >= 10) {
@@ -193,7 +188,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
       const int ksteps = (p.dim + 15) / 16;
       auto scores = [&](int j) {
         const int st = j % kStages, buf = (j - ta) & 1;
-        mbar_wait(smem_u32(&b_full[st]), (j / kStages) & 1, abort_flag, p.status);
+        bar_wait(&b_full[st], (j / kStages) & 1, abort_flag, p.status);
         tc_fence_after();
         const uint32_t a = desc_lo(s_q + g * ks * kSlabQ), b = desc_lo(s_k + st * ks * kSlab);
         for (int k = 0; k < ksteps; ++k) {
@@ -202,10 +197,11 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
         }
         umma_commit(smem_u32(&b_s[g][buf]));
       };
+      bar_wait(&b_q, 0, abort_flag, p.status);
       for (int j = 0; j < tiles; ++j) {
         const int st = j % kStages;
         if (j < ta || j >= tb) {
-          mbar_wait(smem_u32(&b_full[st]), (j / kStages) & 1, abort_flag, p.status);
+          bar_wait(&b_full[st], (j / kStages) & 1, abort_flag, p.status);
           mbar_arrive(smem_u32(&b_empty[st]));
           continue;
         }
@@ -214,7 +210,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
           if (j + 1 < tb) scores(j + 1);
         }
         const int n = j - ta, buf = n & 1;
-        mbar_wait(smem_u32(&b_p[g][buf]), (n >> 1) & 1, abort_flag, p.status);
+        bar_wait(&b_p[g][buf], (n >> 1) & 1, abort_flag, p.status);
         tc_fence_after();
         const uint32_t b = desc_lo_mn(s_v + st * vs * kSlab), pw = t_s + buf * 64;
 #pragma unroll
@@ -231,9 +227,21 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
   } else if (warp >= 8) {
     // ---- copies ----
     const int t = tid - 256, c = t & 15;
+    if (t == 0) {
+      const uint32_t bar = smem_u32(&b_q);
+      if (q_tma) {
+        mbar_expect_tx(bar, 2 * ks * kSlabQ);
+        for (int i = 0; i < 2 * ks; ++i)                          // two boxes of 64 rows fill a slab
+          for (int half = 0; half < 2; ++half)
+            tma_load_2d(s_q + i * kSlabQ + half * (kSlabQ / 2), &map, head * p.dim + (i % ks) * 64,
+                        q0 + m0 + (i / ks) * kTileM + half * 64, bar);
+      } else {
+        mbar_arrive(bar);
+      }
+    }
     for (int j = 0; j < tiles; ++j) {
       const int st = j % kStages, key0 = first + j * kTileKeys;
-      mbar_wait(smem_u32(&b_empty[st]), ((j / kStages) & 1) ^ 1, abort_flag, p.status);
+      bar_wait(&b_empty[st], ((j / kStages) & 1) ^ 1, abort_flag, p.status);
       const uint32_t dk = s_k + st * ks * kSlab, dv = s_v + st * vs * kSlab, full = smem_u32(&b_full[st]);
       if (key0 >= ctx && key0 + kTileKeys <= end) {
         if (t == 0) {
@@ -269,8 +277,28 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
       fence_proxy_async();
       mbar_arrive(full);
     }
-  } else if (rows > 0) {
+  } else {
     // ---- softmax ----
+    if (!q_tma) {
+      const int c = tid & 15;
+      if (c < p.dim / 8) {
+        for (int i = tid >> 4; i < 2 * kTileM; i += 16) {
+          const bool ok = m0 + i < qn;
+          const T* src = qkv + (size_t)(q0 + (ok ? m0 + i : 0)) * p.row_stride + (size_t)head * p.dim + c * 8;
+          cp_async16_u32(s_q + (i >> 7) * ks * kSlabQ + swizzled(i & 127, c, kSlabQ), src, ok);
+        }
+      }
+      cp_async_commit();
+      cp_async_wait<0>();
+      fence_proxy_async();
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(smem_u32(&b_q));
+    for (int i = tid; i < blen + 2 * kBiasPad; i += 256) {
+      const int d = i - kBiasPad;
+      s_bias[i] = d < 0 ? -INFINITY : p.bias ? p.bias[(size_t)head * p.bias_len + min(d, blen - 1)] * kLog2e : 0.f;
+    }
+    named_bar_sync(1, 256);
     const int r = (warp & 3) * 32 + lane, pos = w0 + r;
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t t_o = tmem + 256 + g * 128 + lane_addr;
@@ -279,7 +307,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
     for (int j = ta; j < tb; ++j) {
       const int n = j - ta, buf = n & 1;
       const uint32_t t_s = tmem + g * 128 + buf * 64 + lane_addr;
-      mbar_wait(smem_u32(&b_s[g][buf]), (n >> 1) & 1, abort_flag, p.status);
+      bar_wait(&b_s[g][buf], (n >> 1) & 1, abort_flag, p.status);
       tc_fence_after();
       float s[kTileKeys];
 #pragma unroll
@@ -336,7 +364,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
       }
       l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
       if (rescale) {
-        if (n > 0) mbar_wait(smem_u32(&b_pv[g]), (n - 1) & 1, abort_flag, p.status);   // O holds the products so far
+        if (n > 0) bar_wait(&b_pv[g], (n - 1) & 1, abort_flag, p.status);   // O holds the products so far
         tc_fence_after();
         for (int c = 0; c < vs * 64; c += 32) {
           float o[32];
@@ -350,9 +378,10 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
       }
       tmem_wait_st();
       tc_fence_before();
-      mbar_arrive(smem_u32(&b_p[g][buf]));
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&b_p[g][buf]));
     }
-    mbar_wait(smem_u32(&b_o[g]), 0, abort_flag, p.status);
+    if (tb > ta) bar_wait(&b_o[g], 0, abort_flag, p.status);
     tc_fence_after();
     const float inv = 1.f / l;
     T* op = (T*)p.out + (size_t)(q0 + m0 + g * kTileM + r) * p.heads * p.vdim + (size_t)head * p.vdim + v0;
