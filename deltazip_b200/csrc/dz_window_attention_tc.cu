@@ -45,12 +45,36 @@ __device__ __forceinline__ uint32_t swizzled(int r, int c, int slab) {
   return (uint32_t)((c >> 3) * slab + r * 128 + (((c & 7) ^ (r & 7)) << 4));
 }
 
+// Pairs of 32-bit operations in one instruction.
+struct Pair {
+  unsigned long long v;
+  __device__ __forceinline__ Pair() {}
+  __device__ __forceinline__ Pair(float a, float b) {
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+  }
+  __device__ __forceinline__ void get(float& a, float& b) const {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+  }
+};
+__device__ __forceinline__ Pair fma2(Pair a, Pair b, Pair c) {
+  Pair d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return d;
+}
+__device__ __forceinline__ Pair add2(Pair a, Pair b) {
+  Pair d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d.v) : "l"(a.v), "l"(b.v));
+  return d;
+}
+
 // Two weights as hi + lo pairs.  bf16: hi is the upper half of the float as it stands, lo the rounded rest.
 template <typename T> __device__ __forceinline__ void split_weights(float a, float b, uint32_t& hi, uint32_t& lo) {
   if constexpr (std::is_same<T, __nv_bfloat16>::value) {
     const uint32_t ua = __float_as_uint(a), ub = __float_as_uint(b);
     hi = __byte_perm(ua, ub, 0x7632);
-    lo = Cvt<T>::down(a - __uint_as_float(ua & 0xffff0000u), b - __uint_as_float(ub & 0xffff0000u));
+    float ra, rb;
+    fma2(Pair(__uint_as_float(ua & 0xffff0000u), __uint_as_float(ub & 0xffff0000u)), Pair(-1.f, -1.f), Pair(a, b)).get(ra, rb);
+    lo = Cvt<T>::down(ra, rb);
   } else {
     split_pair<T>(a, b, hi, lo);
   }
@@ -320,13 +344,13 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
         mul = scale2;                                // every distance is in the last column, all keys visible
         add = far_bias;
       } else {                                       // the table holds minus infinity at negative distances
-        const float* tab = s_bias + kBiasPad;
         if (w0 - (t0 + kTileKeys - 1) >= blen - 1) {
 #pragma unroll
           for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, far_bias);
         } else {
+          const float* tab = s_bias + kBiasPad + (pos - t0);
 #pragma unroll
-          for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, tab[pos - t0 - c]);
+          for (int c = 0; c < kTileKeys; ++c) s[c] = fmaf(s[c], scale2, tab[-c]);
         }
         if (cut) {
           const int out = pos - p.window - t0;       // keys up to here have left the window
@@ -348,21 +372,26 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
       }
       const bool rescale = __any_sync(0xffffffffu, f != 1.f);
       add -= m == -INFINITY ? 0.f : m;
-      float sum[4] = {0.f, 0.f, 0.f, 0.f};
+      const Pair mul2(mul, mul), add2v(add, add);
+      Pair sum[2] = {Pair(0.f, 0.f), Pair(0.f, 0.f)};
 #pragma unroll
       for (int c = 0; c < kTileKeys; c += 32) {
         uint32_t hi[16], low[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float a = ex2(fmaf(s[c + 2 * i], mul, add)), b = ex2(fmaf(s[c + 2 * i + 1], mul, add));
-          sum[(2 * i) & 3] += a;
-          sum[(2 * i + 1) & 3] += b;
+          float a, b;
+          fma2(Pair(s[c + 2 * i], s[c + 2 * i + 1]), mul2, add2v).get(a, b);
+          a = ex2(a);
+          b = ex2(b);
+          sum[i & 1] = add2(sum[i & 1], Pair(a, b));
           split_weights<T>(a, b, hi[i], low[i]);
         }
         tmem_st16(t_s + c / 2, hi);
         tmem_st16(t_s + 32 + c / 2, low);
       }
-      l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
+      float la, lb;
+      add2(sum[0], sum[1]).get(la, lb);
+      l += la + lb;
       if (rescale) {
         if (n > 0) bar_wait(&b_pv[g], (n - 1) & 1, abort_flag, p.status);   // O holds the products so far
         tc_fence_after();
