@@ -53,7 +53,7 @@ __device__ __forceinline__ float soft_cap(float x, float cap) { return cap * tan
 constexpr int kRecThreads = 256, kRowsInFlight = 8;
 
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kRecThreads)
+__global__ void __launch_bounds__(kRecThreads, 3)
 mlstm_recurrent_kernel(MlstmParams p, int vt) {
   extern __shared__ float sm[];
   __shared__ float s_part[kRecThreads / 32], s_part2[kRecThreads / 32];
@@ -79,10 +79,31 @@ mlstm_recurrent_kernel(MlstmParams p, int vt) {
   const T* wi = (const T*)p.w_if + (size_t)head * p.width;
   const T* wf = (const T*)p.w_if + (size_t)(p.heads + head) * p.width;
 
+  // rows d0, d0 + rg_n, ... of this thread's columns of S (zero where there are none)
+  float s[kRowsInFlight][VEC];
+  auto load_rows = [&](int d0, bool zero) {
+#pragma unroll
+    for (int u = 0; u < kRowsInFlight; ++u) {
+      const int d = d0 + u * rg_n;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) s[u][j] = 0.f;
+      if (mine && d < p.dim && !zero) {
+        const float* src = S + (size_t)d * p.vdim + cgi * VEC;
+        if constexpr (VEC == 4) {
+          const float4 x = *reinterpret_cast<const float4*>(src);
+          s[u][0] = x.x; s[u][1] = x.y; s[u][2] = x.z; s[u][3] = x.w;
+        } else {
+          s[u][0] = *src;
+        }
+      }
+    }
+  };
+
   for (int t = 0; t < tn; ++t) {
     const T* row = (const T*)p.x + (size_t)(q0 + t) * p.row_stride;
     const T* h = (const T*)p.h + (size_t)(q0 + t) * p.width;
     const bool zero = ctx == 0 && t == 0;           // the state before this token is zero
+    load_rows(rgi, zero);                           // on their way while the gates are computed
     for (int d = tid; d < p.dim; d += kRecThreads) {
       sq[d] = Cvt<T>::one(row[(size_t)head * p.dim + d]) * p.scale;
       sk[d] = Cvt<T>::one(row[p.k_off + (size_t)head * p.dim + d]);
@@ -132,22 +153,7 @@ mlstm_recurrent_kernel(MlstmParams p, int vt) {
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v[j] = sv[cgi * VEC + j] * add;
       for (int d0 = rgi; d0 < p.dim; d0 += rg_n * kRowsInFlight) {
-        float s[kRowsInFlight][VEC];
-#pragma unroll
-        for (int u = 0; u < kRowsInFlight; ++u) {
-          const int d = d0 + u * rg_n;
-#pragma unroll
-          for (int j = 0; j < VEC; ++j) s[u][j] = 0.f;
-          if (d < p.dim && !zero) {
-            const float* src = S + (size_t)d * p.vdim + cgi * VEC;
-            if constexpr (VEC == 4) {
-              const float4 x = *reinterpret_cast<const float4*>(src);
-              s[u][0] = x.x; s[u][1] = x.y; s[u][2] = x.z; s[u][3] = x.w;
-            } else {
-              s[u][0] = *src;
-            }
-          }
-        }
+        if (d0 != rgi) load_rows(d0, zero);
 #pragma unroll
         for (int u = 0; u < kRowsInFlight; ++u) {
           const int d = d0 + u * rg_n;
@@ -208,24 +214,25 @@ mlstm_recurrent_kernel(MlstmParams p, int vt) {
 // and M_t = max(m_start, max_{s <= t} a_s), m_t = F_t + M_t and
 //   o_t ~ sum_{s <= t} e^(a_s - M_t) (q_t.k_s) v_s + e^(m_start - M_t) q_t S_start
 //   S_end = e^(m_start - M_L) S_start + sum_s e^(a_s - M_L) k_s v_s^T.
-// A CTA of four warps owns VT value columns of one (head, sequence) and walks the chunks; its slice
+// A CTA of eight warps owns VT value columns of one (head, sequence) and walks the chunks; its slice
 // of S stays in shared memory in 32 bits, transposed, with n as one more row (the value matrix gets
 // a column of ones).  32-bit operands enter the MMAs as hi + lo pairs.  Writes the cell's output before the
 // head norm.  Grid (tiles of VT columns, heads, sequences).
 // -------------------------------------------------------------------------------------------------
-constexpr int kL = 64;
+constexpr int kL = 64, kChunkThreads = 256;
 
 template <int VT> __host__ __device__ constexpr int chunk_ldv() { return VT + 24; }
 
 template <typename T, int VT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kChunkThreads)
 mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
-  constexpr int NT = VT / 8, LDV = chunk_ldv<VT>();
+  constexpr int NT = VT / 16, LDV = chunk_ldv<VT>();   // a warp: 16 rows, half of the columns
   extern __shared__ uint4 smem_raw[];
   __shared__ float s_a[kL], s_mx[kL], s_inter[kL], s_em[kL], s_w[kL];
   __shared__ float s_m, s_decay, s_mnext;
   __shared__ int s_last;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int rw = warp & 3, cw = (warp >> 2) * (VT / 2);
   const int head = blockIdx.y, seq = blockIdx.z, v0 = blockIdx.x * VT;
   pdl_wait();
   pdl_launch();
@@ -242,20 +249,34 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
   float* gn = p.n + ((size_t)slot * p.heads + head) * p.dim;
   float* gm = p.m + (size_t)slot * p.heads + head;
   const int bytes = kL * (2 * ldk + LDV) * 2 + (VT + 16) * lds * 4;
-  for (int i = tid; i < bytes / 16; i += 128) smem_raw[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < bytes / 16; i += kChunkThreads) smem_raw[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
-  for (int i = tid; i < kL; i += 128) sv[i * LDV + VT] = Cvt<T>::from(1.f);
+  for (int i = tid; i < kL; i += kChunkThreads) sv[i * LDV + VT] = Cvt<T>::from(1.f);
   if (ctx > 0) {
-    for (int i = tid; i < p.dim * VT; i += 128) {
+    for (int i = tid; i < p.dim * VT; i += kChunkThreads) {
       const int d = i / VT, c = i % VT;
       if (c < vcols) st[c * lds + d] = S[(size_t)d * p.vdim + c];
     }
-    for (int d = tid; d < p.dim; d += 128) st[VT * lds + d] = gn[d];
+    for (int d = tid; d < p.dim; d += kChunkThreads) st[VT * lds + d] = gn[d];
   }
   if (tid == 0) s_m = ctx > 0 ? *gm : 0.f;
   const T* x = (const T*)p.x;
-  const int r = tid >> 1, c0 = tid & 1;
+  const int r = tid >> 2, c0 = tid & 3;
   bool have_state = ctx > 0;
+  // gate pre-activations of a chunk (warp 0; lane l holds tokens 2l and 2l + 1), fetched a chunk ahead
+  float pi[2], pf[2];
+  auto fetch_gates = [&](int base) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int t = base + 2 * lane + j;
+      if (warp == 0 && t < qn) {
+        const float* pre = p.pre_if + (size_t)(q0 + t) * 2 * p.heads;
+        pi[j] = pre[head];
+        pf[j] = pre[p.heads + head];
+      }
+    }
+  };
+  fetch_gates(0);
   __syncthreads();
 
   for (int base = 0; base < qn; base += kL) {
@@ -266,14 +287,14 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
       const T* qs = row + (size_t)head * p.dim;
       const T* ks = row + p.k_off + (size_t)head * p.dim;
       const T* vs = row + p.v_off + (size_t)head * p.vdim + v0;
-      for (int c = c0; c < p.dim / 8; c += 2) {
+      for (int c = c0; c < p.dim / 8; c += 4) {
         cp_async16(sq + r * ldk + c * 8, qs + c * 8, ok);
         cp_async16(sk + r * ldk + c * 8, ks + c * 8, ok);
       }
-      for (int c = c0; c < vcols / 8; c += 2) cp_async16(sv + r * LDV + c * 8, vs + c * 8, ok);
+      for (int c = c0; c < vcols / 8; c += 4) cp_async16(sv + r * LDV + c * 8, vs + c * 8, ok);
       cp_async_commit();
     }
-    if (warp == 0) {                                 // gates: lane l holds tokens 2l and 2l + 1
+    if (warp == 0) {                                 // gates
       float gi[2], gf[2];
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
@@ -281,9 +302,8 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
         gi[j] = -INFINITY;                           // absent tokens add nothing and forget nothing
         gf[j] = 0.f;
         if (t < len) {
-          const float* pre = p.pre_if + (size_t)(q0 + base + t) * 2 * p.heads;
-          gi[j] = soft_cap(pre[head] + p.b_if[head], p.cap);
-          gf[j] = log_sigmoid(soft_cap(pre[p.heads + head] + p.b_if[p.heads + head], p.cap));
+          gi[j] = soft_cap(pi[j] + p.b_if[head], p.cap);
+          gf[j] = log_sigmoid(soft_cap(pf[j] + p.b_if[p.heads + head], p.cap));
         }
       }
       float f = gf[0] + gf[1];
@@ -313,11 +333,12 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
       s_w[t] = expf(a0 - ML); s_w[t + 1] = expf(a1 - ML);
       if (lane == 0) { s_decay = expf(m0 - ML); s_mnext = FL + ML; }
     }
+    fetch_gates(base + kL);
     cp_async_wait<0>();
     __syncthreads();
 
-    const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
-    if (warp * 16 < len) {
+    const int r0 = rw * 16 + (lane >> 2), r1 = r0 + 8;
+    if (rw * 16 < len) {
       float o[NT + 1][4];
 #pragma unroll
       for (int i = 0; i <= NT; ++i)
@@ -328,14 +349,14 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
       for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
-      const T* aq = sq + (warp * 16 + (lane & 15)) * ldk + (lane >> 4) * 8;
+      const T* aq = sq + (rw * 16 + (lane & 15)) * ldk + (lane >> 4) * 8;
       const T* bk = sk + ((lane & 7) + ((lane >> 4) & 1) * 8) * ldk + ((lane >> 3) & 1) * 8;
       for (int kk = 0; kk < dimp; kk += 16) {
         uint32_t a[4];
         ldsm4(a, aq + kk);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          if (j <= warp) {                           // keys up to the warp's last row
+          if (j <= rw) {                             // keys up to the warp's last row
             uint32_t b[4];
             ldsm4(b, bk + j * 16 * ldk + kk);
             mma16816<T>(s[2 * j], a, b[0], b[1]);
@@ -343,16 +364,18 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
           }
         }
         if (have_state) {
+          uint32_t bh[NT + 1][2], bl[NT + 1][2];
 #pragma unroll
-          for (int i = 0; i <= NT; ++i) {
-            const float* sp = st + (i * 8 + (lane >> 2)) * lds + kk + (lane & 3) * 2;
+          for (int i = 0; i <= NT; ++i) {           // the last tile holds n
+            const float* sp = st + ((i < NT ? cw + i * 8 : VT) + (lane >> 2)) * lds + kk + (lane & 3) * 2;
             const float2 x0 = *reinterpret_cast<const float2*>(sp), x1 = *reinterpret_cast<const float2*>(sp + 8);
-            uint32_t h0, l0, h1, l1;
-            split_pair<T>(x0.x, x0.y, h0, l0);
-            split_pair<T>(x1.x, x1.y, h1, l1);
-            mma16816<T>(o[i], a, h0, h1);
-            mma16816<T>(o[i], a, l0, l1);
+            split_pair<T>(x0.x, x0.y, bh[i][0], bl[i][0]);
+            split_pair<T>(x1.x, x1.y, bh[i][1], bl[i][1]);
           }
+#pragma unroll
+          for (int i = 0; i <= NT; ++i) mma16816<T>(o[i], a, bh[i][0], bh[i][1]);
+#pragma unroll
+          for (int i = 0; i <= NT; ++i) mma16816<T>(o[i], a, bl[i][0], bl[i][1]);
         }
       }
       const float in0 = s_inter[r0], in1 = s_inter[r1], mx0 = s_mx[r0], mx1 = s_mx[r1];
@@ -374,7 +397,7 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
       const T* bv = sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * LDV + ((lane >> 4) & 1) * 8;
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
-        if (kk <= warp) {
+        if (kk <= rw) {
           uint32_t hi[4], lo[4];
           split_pair<T>(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
           split_pair<T>(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
@@ -383,7 +406,7 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
 #pragma unroll
           for (int i = 0; i < NT; i += 2) {
             uint32_t b[4];
-            ldsm4_t(b, bv + kk * 16 * LDV + i * 8);
+            ldsm4_t(b, bv + kk * 16 * LDV + cw + i * 8);
             mma16816<T>(o[i], hi, b[0], b[1]);
             mma16816<T>(o[i + 1], hi, b[2], b[3]);
             mma16816<T>(o[i], lo, b[0], b[1]);
@@ -402,7 +425,7 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
       T* op = (T*)p.out + (size_t)(q0 + base) * p.heads * p.vdim + (size_t)head * p.vdim + v0;
 #pragma unroll
       for (int i = 0; i < NT; ++i) {
-        const int c = i * 8 + (lane & 3) * 2;
+        const int c = cw + i * 8 + (lane & 3) * 2;
         if (c < vcols) {
           if (r0 < len)
             *reinterpret_cast<uint32_t*>(op + (size_t)r0 * p.heads * p.vdim + c) = Cvt<T>::down(o[i][0] * d0, o[i][1] * d0);
@@ -428,7 +451,7 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
           split_pair<T>(f.x * s_w[o], f.y * s_w[o + 1], hi[kk][j], lo[kk][j]);
         }
       }
-      for (int nt = warp; nt < dimp / 8; nt += 4) {
+      for (int nt = warp; nt < dimp / 8; nt += kChunkThreads / 32) {
         float* c0p = st + (mt * 16 + (lane >> 2)) * lds + nt * 8 + (lane & 3) * 2;
         float* c1p = c0p + 8 * lds;
         const float2 x0 = *reinterpret_cast<const float2*>(c0p), x1 = *reinterpret_cast<const float2*>(c1p);
@@ -450,7 +473,7 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
     have_state = true;
     __syncthreads();
   }
-  for (int i = tid; i < p.dim * VT; i += 128) {
+  for (int i = tid; i < p.dim * VT; i += kChunkThreads) {
     const int d = i / VT, c = i % VT;
     if (c < vcols) S[(size_t)d * p.vdim + c] = st[c * lds + d];
   }
@@ -464,7 +487,7 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
   }
   __syncthreads();
   if (s_last) {
-    for (int d = tid; d < p.dim; d += 128) gn[d] = st[VT * lds + d];
+    for (int d = tid; d < p.dim; d += kChunkThreads) gn[d] = st[VT * lds + d];
     if (tid == 0) *gm = s_m;
   }
 }
@@ -521,7 +544,7 @@ template <typename T, int VT>
 int run_chunk(const MlstmParams& p, int num_seqs, int dimp, int* tickets, cudaStream_t st) {
   const size_t smem = chunk_smem(dimp, VT);
   DZ_CUDA_OK(allow_smem(mlstm_chunk_kernel<T, VT>, smem));
-  DZ_CUDA_OK(launch_ex(mlstm_chunk_kernel<T, VT>, dim3((p.vdim + VT - 1) / VT, p.heads, num_seqs), dim3(128), smem, 1,
+  DZ_CUDA_OK(launch_ex(mlstm_chunk_kernel<T, VT>, dim3((p.vdim + VT - 1) / VT, p.heads, num_seqs), dim3(kChunkThreads), smem, 1,
                        st, p, dimp, tickets));
   return DZ_OK;
 }
@@ -530,9 +553,9 @@ template <typename T>
 int run_recurrent(const MlstmParams& p, int num_seqs, cudaStream_t st) {
   const bool vec = p.vdim % 4 == 0 && p.width % 8 == 0 && aligned16(p.h) && aligned16(p.w_if) && aligned16(p.S);
   const int v = vec ? 4 : 1;
-  // columns per CTA: a slice of S of about 32 KB, at most 8 CTAs (and never more column groups than threads)
+  // columns per CTA: a slice of S of at most 64 KB, at most 8 CTAs (and never more column groups than threads)
   int c = 1;
-  while (c < 8 && (size_t)p.dim * ((p.vdim + c - 1) / c) * 4 > 32 * 1024 && p.vdim / (2 * c) >= v) c *= 2;
+  while (c < 8 && (size_t)p.dim * ((p.vdim + c - 1) / c) * 4 > 64 * 1024 && p.vdim / (2 * c) >= v) c *= 2;
   int vt = ((p.vdim + c - 1) / c + v - 1) / v * v;
   while (vt / v > kRecThreads && c < 8) { c *= 2; vt = ((p.vdim + c - 1) / c + v - 1) / v * v; }
   const int rg = kRecThreads / (vt / v > 0 ? vt / v : 1);
