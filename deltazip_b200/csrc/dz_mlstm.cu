@@ -215,18 +215,20 @@ mlstm_recurrent_kernel(MlstmParams p, int vt) {
 //   o_t ~ sum_{s <= t} e^(a_s - M_t) (q_t.k_s) v_s + e^(m_start - M_t) q_t S_start
 //   S_end = e^(m_start - M_L) S_start + sum_s e^(a_s - M_L) k_s v_s^T.
 // A CTA of eight warps owns VT value columns of one (head, sequence) and walks the chunks; its slice
-// of S stays in shared memory in 32 bits, transposed, with n as one more row (the value matrix gets
-// a column of ones).  32-bit operands enter the MMAs as hi + lo pairs.  Writes the cell's output before the
+// of S stays in registers in 32 bits, as accumulators of the update, with n as one more row (the value
+// matrix gets a column of ones).  32-bit operands enter the MMAs as hi + lo pairs, split once: S after
+// its update, v times its gate weight at the start of a chunk.  A warp owns NTW groups of eight rows of
+// k's columns (64 NTW >= dim).  Writes the cell's output before the
 // head norm.  Grid (tiles of VT columns, heads, sequences).
 // -------------------------------------------------------------------------------------------------
 constexpr int kL = 64, kChunkThreads = 256;
 
 template <int VT> __host__ __device__ constexpr int chunk_ldv() { return VT + 24; }
 
-template <typename T, int VT>
-__global__ void __launch_bounds__(kChunkThreads)
+template <typename T, int VT, int NTW>
+__global__ void __launch_bounds__(kChunkThreads, 1)
 mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
-  constexpr int NT = VT / 16, LDV = chunk_ldv<VT>();   // a warp: 16 rows, half of the columns
+  constexpr int NT = VT / 16, MT = VT / 16 + 1, LDV = chunk_ldv<VT>();   // output: a warp has 16 rows, half of the columns
   extern __shared__ uint4 smem_raw[];
   __shared__ float s_a[kL], s_mx[kL], s_inter[kL], s_em[kL], s_w[kL];
   __shared__ float s_m, s_decay, s_mnext;
@@ -244,20 +246,55 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
   T* sq = reinterpret_cast<T*>(smem_raw);
   T* sk = sq + kL * ldk;
   T* sv = sk + kL * ldk;
-  float* st = reinterpret_cast<float*>(sv + kL * LDV);            // [VT + 16][lds]
+  T* wh = sv + kL * LDV;                                          // v times its gate weight, hi and lo
+  T* wl = wh + kL * LDV;
+  T* sh = wl + kL * LDV;                                          // S transposed, hi and lo: [VT + 16][lds]
+  T* sl = sh + (VT + 16) * lds;
   float* S = p.S + ((size_t)slot * p.heads + head) * p.dim * p.vdim + v0;
   float* gn = p.n + ((size_t)slot * p.heads + head) * p.dim;
   float* gm = p.m + (size_t)slot * p.heads + head;
-  const int bytes = kL * (2 * ldk + LDV) * 2 + (VT + 16) * lds * 4;
+  const int bytes = kL * (2 * ldk + 3 * LDV) * 2 + 2 * (VT + 16) * lds * 2;
   for (int i = tid; i < bytes / 16; i += kChunkThreads) smem_raw[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
   for (int i = tid; i < kL; i += kChunkThreads) sv[i * LDV + VT] = Cvt<T>::from(1.f);
+  // The state itself: rows mt * 16 + lane / 4 (+ 8), columns nt * 8 + 2 (lane % 4) (+ 1) of the transposed
+  // slice, nt = warp + 8 i; the first row past the value columns is n.
+  float acc[MT][NTW][4];
+  const int col0 = warp * 8 + (lane & 3) * 2;
+  auto each = [&](auto&& fn) {                       // fn(value, dim index, value column or -1 for n)
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int i = 0; i < NTW; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = col0 + i * 64 + (e & 1), v = mt * 16 + (lane >> 2) + (e >> 1) * 8;
+          if (d < p.dim && (mt < MT - 1 ? v < vcols : v == VT)) fn(acc[mt][i][e], d, mt < MT - 1 ? v : -1);
+        }
+  };
+  auto publish = [&]() {
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int i = 0; i < NTW; ++i)
+        if (warp + 8 * i < dimp / 8) {
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const int at = (mt * 16 + (lane >> 2) + e * 4) * lds + col0 + i * 64;
+            split_pair<T>(acc[mt][i][e], acc[mt][i][e + 1], *reinterpret_cast<uint32_t*>(sh + at),
+                          *reinterpret_cast<uint32_t*>(sl + at));
+          }
+        }
+  };
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int i = 0; i < NTW; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[mt][i][e] = 0.f;
   if (ctx > 0) {
-    for (int i = tid; i < p.dim * VT; i += kChunkThreads) {
-      const int d = i / VT, c = i % VT;
-      if (c < vcols) st[c * lds + d] = S[(size_t)d * p.vdim + c];
-    }
-    for (int d = tid; d < p.dim; d += kChunkThreads) st[VT * lds + d] = gn[d];
+    each([&](float& x, int d, int v) { x = v < 0 ? gn[d] : S[(size_t)d * p.vdim + v]; });
+    publish();
   }
   if (tid == 0) s_m = ctx > 0 ? *gm : 0.f;
   const T* x = (const T*)p.x;
@@ -336,6 +373,12 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
     fetch_gates(base + kL);
     cp_async_wait<0>();
     __syncthreads();
+    for (int i = tid; i < kL * (VT + 16) / 2; i += kChunkThreads) {
+      const int t = i / ((VT + 16) / 2), at = t * LDV + 2 * (i % ((VT + 16) / 2));
+      const float2 f = Cvt<T>::up(*reinterpret_cast<const uint32_t*>(sv + at));
+      const float w = s_w[t];
+      split_pair<T>(f.x * w, f.y * w, *reinterpret_cast<uint32_t*>(wh + at), *reinterpret_cast<uint32_t*>(wl + at));
+    }
 
     const int r0 = rw * 16 + (lane >> 2), r1 = r0 + 8;
     if (rw * 16 < len) {
@@ -364,18 +407,18 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
           }
         }
         if (have_state) {
-          uint32_t bh[NT + 1][2], bl[NT + 1][2];
+          uint32_t bh[NT / 2 + 1][4], bl[NT / 2 + 1][4];
 #pragma unroll
-          for (int i = 0; i <= NT; ++i) {           // the last tile holds n
-            const float* sp = st + ((i < NT ? cw + i * 8 : VT) + (lane >> 2)) * lds + kk + (lane & 3) * 2;
-            const float2 x0 = *reinterpret_cast<const float2*>(sp), x1 = *reinterpret_cast<const float2*>(sp + 8);
-            split_pair<T>(x0.x, x0.y, bh[i][0], bl[i][0]);
-            split_pair<T>(x1.x, x1.y, bh[i][1], bl[i][1]);
+          for (int i = 0; i <= NT / 2; ++i) {       // the last pair of tiles starts with n
+            const int at = ((i < NT / 2 ? cw + i * 16 : VT) + (lane & 7) + ((lane >> 4) & 1) * 8) * lds +
+                           ((lane >> 3) & 1) * 8 + kk;
+            ldsm4(bh[i], sh + at);
+            ldsm4(bl[i], sl + at);
           }
 #pragma unroll
-          for (int i = 0; i <= NT; ++i) mma16816<T>(o[i], a, bh[i][0], bh[i][1]);
+          for (int i = 0; i <= NT; ++i) mma16816<T>(o[i], a, bh[i / 2][2 * (i & 1)], bh[i / 2][2 * (i & 1) + 1]);
 #pragma unroll
-          for (int i = 0; i <= NT; ++i) mma16816<T>(o[i], a, bl[i][0], bl[i][1]);
+          for (int i = 0; i <= NT; ++i) mma16816<T>(o[i], a, bl[i / 2][2 * (i & 1)], bl[i / 2][2 * (i & 1) + 1]);
         }
       }
       const float in0 = s_inter[r0], in1 = s_inter[r1], mx0 = s_mx[r0], mx1 = s_mx[r1];
@@ -436,47 +479,46 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
     }
     __syncthreads();                                 // the old state has been read
     const float decay = s_decay;
-#pragma unroll 1
-    for (int mt = 0; mt <= VT / 16; ++mt) {          // 16 value columns, or the column of ones
-      uint32_t hi[4][4], lo[4][4];
+    uint32_t kb[NTW][8];                             // this warp's columns of k, all 64 tokens
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk) {
-        uint32_t a[4];
-        ldsm4_t(a, sv + (kk * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * LDV + mt * 16 + ((lane >> 3) & 1) * 8);
-        const int t = kk * 16 + (lane & 3) * 2;
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float2 f = Cvt<T>::up(a[j]);
-          const int o = t + (j >> 1) * 8;
-          split_pair<T>(f.x * s_w[o], f.y * s_w[o + 1], hi[kk][j], lo[kk][j]);
-        }
-      }
-      for (int nt = warp; nt < dimp / 8; nt += kChunkThreads / 32) {
-        float* c0p = st + (mt * 16 + (lane >> 2)) * lds + nt * 8 + (lane & 3) * 2;
-        float* c1p = c0p + 8 * lds;
-        const float2 x0 = *reinterpret_cast<const float2*>(c0p), x1 = *reinterpret_cast<const float2*>(c1p);
-        float c[4] = {x0.x * decay, x0.y * decay, x1.x * decay, x1.y * decay};
+    for (int i = 0; i < NTW; ++i)
+      if (warp + 8 * i < dimp / 8) {
+        uint32_t b[4];
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          uint32_t b[4];
-          ldsm4_t(b, sk + (j * 32 + lane) * ldk + nt * 8);
-          mma16816<T>(c, hi[2 * j], b[0], b[1]);
-          mma16816<T>(c, lo[2 * j], b[0], b[1]);
-          mma16816<T>(c, hi[2 * j + 1], b[2], b[3]);
-          mma16816<T>(c, lo[2 * j + 1], b[2], b[3]);
+          ldsm4_t(b, sk + (j * 32 + lane) * ldk + (warp + 8 * i) * 8);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) kb[i][4 * j + e] = b[e];
         }
-        *reinterpret_cast<float2*>(c0p) = make_float2(c[0], c[1]);
-        *reinterpret_cast<float2*>(c1p) = make_float2(c[2], c[3]);
+      }
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {                // 16 value columns, or the column of ones
+#pragma unroll
+      for (int i = 0; i < NTW; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[mt][i][e] *= decay;
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        uint32_t hi[4], lo[4];
+        const int at = (kk * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * LDV + mt * 16 + ((lane >> 3) & 1) * 8;
+        ldsm4_t(hi, wh + at);
+        ldsm4_t(lo, wl + at);
+#pragma unroll
+        for (int i = 0; i < NTW; ++i)
+          if (warp + 8 * i < dimp / 8) mma16816<T>(acc[mt][i], hi, kb[i][2 * kk], kb[i][2 * kk + 1]);
+#pragma unroll
+        for (int i = 0; i < NTW; ++i)
+          if (warp + 8 * i < dimp / 8) mma16816<T>(acc[mt][i], lo, kb[i][2 * kk], kb[i][2 * kk + 1]);
       }
     }
+    publish();
     if (tid == 0) s_m = s_mnext;
     have_state = true;
     __syncthreads();
   }
-  for (int i = tid; i < p.dim * VT; i += kChunkThreads) {
-    const int d = i / VT, c = i % VT;
-    if (c < vcols) S[(size_t)d * p.vdim + c] = st[c * lds + d];
-  }
+  each([&](float& x, int d, int v) {
+    if (v >= 0) S[(size_t)d * p.vdim + v] = x;
+  });
   // n and m, read by every CTA of this (head, sequence) at its start, are written by the last to end
   __threadfence();
   __syncthreads();
@@ -487,7 +529,9 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
   }
   __syncthreads();
   if (s_last) {
-    for (int d = tid; d < p.dim; d += kChunkThreads) gn[d] = st[VT * lds + d];
+    each([&](float& x, int d, int v) {
+      if (v < 0) gn[d] = x;
+    });
     if (tid == 0) *gm = s_m;
   }
 }
@@ -537,16 +581,23 @@ head_norm_gate_kernel(const T* o, const T* __restrict__ g, int64_t g_stride, con
 }
 
 size_t chunk_smem(int dimp, int vt) {
-  return (size_t)kL * (2 * (dimp + 8) + vt + 24) * 2 + (size_t)(vt + 16) * (dimp + 8) * 4;
+  return (size_t)kL * (2 * (dimp + 8) + 3 * (vt + 24)) * 2 + (size_t)2 * (vt + 16) * (dimp + 8) * 2;
 }
 
+template <typename T, int VT, int NTW>
+int run_chunk_n(const MlstmParams& p, int num_seqs, int dimp, int* tickets, cudaStream_t st) {
+  const size_t smem = chunk_smem(dimp, VT);
+  DZ_CUDA_OK(allow_smem(mlstm_chunk_kernel<T, VT, NTW>, smem));
+  DZ_CUDA_OK(launch_ex(mlstm_chunk_kernel<T, VT, NTW>, dim3((p.vdim + VT - 1) / VT, p.heads, num_seqs),
+                       dim3(kChunkThreads), smem, 1, st, p, dimp, tickets));
+  return DZ_OK;
+}
 template <typename T, int VT>
 int run_chunk(const MlstmParams& p, int num_seqs, int dimp, int* tickets, cudaStream_t st) {
-  const size_t smem = chunk_smem(dimp, VT);
-  DZ_CUDA_OK(allow_smem(mlstm_chunk_kernel<T, VT>, smem));
-  DZ_CUDA_OK(launch_ex(mlstm_chunk_kernel<T, VT>, dim3((p.vdim + VT - 1) / VT, p.heads, num_seqs), dim3(kChunkThreads), smem, 1,
-                       st, p, dimp, tickets));
-  return DZ_OK;
+  if (dimp <= 64) return run_chunk_n<T, VT, 1>(p, num_seqs, dimp, tickets, st);
+  if (dimp <= 128) return run_chunk_n<T, VT, 2>(p, num_seqs, dimp, tickets, st);
+  if (dimp <= 256) return run_chunk_n<T, VT, 4>(p, num_seqs, dimp, tickets, st);
+  return run_chunk_n<T, 32, 8>(p, num_seqs, dimp, tickets, st);
 }
 
 template <typename T>
@@ -583,7 +634,8 @@ extern "C" {
 int dz_mlstm_chunk_supported(int dim, int vdim, int dtype) {
   if (dtype != DZ_DTYPE_F16 && dtype != DZ_DTYPE_BF16) return 0;
   if (dim <= 0 || vdim <= 0 || dim % 8 || vdim % 8) return 0;
-  return chunk_smem((dim + 15) / 16 * 16, 32) <= kMaxDynSmem;
+  const int dimp = (dim + 15) / 16 * 16;
+  return dimp <= 512 && chunk_smem(dimp, 32) <= kMaxDynSmem;
 }
 
 size_t dz_mlstm_workspace_bytes(int num_seqs, int heads) {
@@ -617,7 +669,7 @@ int dz_mlstm(const dz_mlstm_args* a, void* stream) {
   if (!a->workspace || a->workspace_bytes < dz_mlstm_workspace_bytes(a->num_seqs, a->heads)) return DZ_ERR_WORKSPACE;
   const int dimp = (a->dim + 15) / 16 * 16;
   int rc = DZ_OK;
-  const bool wide = a->vdim > 32 && chunk_smem(dimp, 64) <= kMaxDynSmem;
+  const bool wide = a->vdim > 32 && dimp <= 256 && chunk_smem(dimp, 64) <= kMaxDynSmem;
   DZ_DISPATCH16(a->dtype, rc = wide ? run_chunk<T, 64>(p, a->num_seqs, dimp, (int*)a->workspace, st)
                                     : run_chunk<T, 32>(p, a->num_seqs, dimp, (int*)a->workspace, st));
   if (rc) return rc;
