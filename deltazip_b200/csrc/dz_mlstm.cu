@@ -373,11 +373,16 @@ mlstm_chunk_kernel(MlstmParams p, int dimp, int* __restrict__ tickets) {
     fetch_gates(base + kL);
     cp_async_wait<0>();
     __syncthreads();
-    for (int i = tid; i < kL * (VT + 16) / 2; i += kChunkThreads) {
-      const int t = i / ((VT + 16) / 2), at = t * LDV + 2 * (i % ((VT + 16) / 2));
-      const float2 f = Cvt<T>::up(*reinterpret_cast<const uint32_t*>(sv + at));
-      const float w = s_w[t];
-      split_pair<T>(f.x * w, f.y * w, *reinterpret_cast<uint32_t*>(wh + at), *reinterpret_cast<uint32_t*>(wl + at));
+    for (int i = c0; i < (VT + 16) / 8; i += 4) {     // four threads a row, eight columns at a time
+      const int at = r * LDV + i * 8;
+      const float w = s_w[r];
+      float f[8];
+      load8<T>(sv + at, f);
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) split_pair<T>(f[2 * j] * w, f[2 * j + 1] * w, hi[j], lo[j]);
+      *reinterpret_cast<uint4*>(wh + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(wl + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
 
     const int r0 = rw * 16 + (lane >> 2), r1 = r0 + 8;
