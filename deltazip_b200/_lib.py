@@ -32,6 +32,8 @@ DZ_INDEX_I32 = 0
 DZ_INDEX_I64 = 1
 DZ_ACT_SILU = 0
 DZ_ACT_GELU_TANH = 1
+DZ_ACT_RELU2 = 2
+DZ_ACT_NONE = -1
 DZ_SBMM_ACCUMULATE = 1
 DZ_SBMM_INPUTS_STABLE = 2
 
@@ -68,6 +70,7 @@ class WindowAttentionArgs(Structure):
         ("heads", c_int32), ("kv_heads", c_int32), ("dim", c_int32), ("vdim", c_int32),
         ("scale", c_float), ("window", c_int32), ("bias", c_void_p), ("bias_len", c_int32), ("splits", c_int32),
         ("workspace", c_void_p), ("workspace_bytes", c_size_t), ("dtype", c_int32),
+        ("sink", c_void_p), ("kv", c_void_p), ("kv_stride", c_int64), ("kv_starts", c_void_p), ("kv_rows", c_int32),
     ]
 
 
@@ -81,6 +84,38 @@ class MlstmArgs(Structure):
         ("ctx_lens", c_void_p), ("num_seqs", c_int32), ("rows", c_int32), ("heads", c_int32), ("dim", c_int32),
         ("vdim", c_int32), ("chunkwise", c_int32), ("workspace", c_void_p), ("workspace_bytes", c_size_t),
         ("dtype", c_int32),
+    ]
+
+
+class LatentRowsArgs(Structure):
+    """Mirror of dz_latent_rows_args."""
+    _fields_ = [
+        ("x", c_void_p), ("row_stride", c_int64), ("positions", c_void_p), ("freq", c_void_p), ("rows", c_int32),
+        ("heads", c_int32), ("dim", c_int32), ("rot", c_int32), ("q_out", c_void_p), ("l_off", c_int32),
+        ("rank", c_int32), ("norm_weight", c_void_p), ("eps", c_float), ("cache", c_void_p), ("slots", c_void_p),
+        ("dtype", c_int32),
+    ]
+
+
+class LatentAttentionArgs(Structure):
+    """Mirror of dz_latent_attention_args."""
+    _fields_ = [
+        ("q", c_void_p), ("cache", c_void_p), ("block_tables", c_void_p), ("table_width", c_int32),
+        ("block_size", c_int32), ("q_starts", c_void_p), ("ctx_lens", c_void_p), ("num_seqs", c_int32),
+        ("rows", c_int32), ("heads", c_int32), ("rank", c_int32), ("rot", c_int32), ("scale", c_float),
+        ("sink", c_void_p), ("out", c_void_p), ("splits", c_int32), ("workspace", c_void_p),
+        ("workspace_bytes", c_size_t), ("dtype", c_int32),
+    ]
+
+
+class LightningArgs(Structure):
+    """Mirror of dz_lightning_args."""
+    _fields_ = [
+        ("x", c_void_p), ("row_stride", c_int64), ("k_off", c_int32), ("v_off", c_int32), ("g_off", c_int32),
+        ("powers", c_void_p), ("norm_weight", c_void_p), ("eps", c_float), ("out", c_void_p), ("S", c_void_p),
+        ("slots", c_void_p), ("q_starts", c_void_p), ("ctx_lens", c_void_p), ("num_seqs", c_int32), ("rows", c_int32),
+        ("heads", c_int32), ("dim", c_int32), ("vdim", c_int32), ("chunkwise", c_int32), ("workspace", c_void_p),
+        ("workspace_bytes", c_size_t), ("dtype", c_int32),
     ]
 
 
@@ -131,10 +166,11 @@ _SIGNATURES = {
     "dz_paged_attention_decode": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                                           c_void_p, c_size_t, c_int, c_void_p]),
-    "dz_embed_norm": (c_int, [c_void_p, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p, c_int64, c_int,
+    "dz_embed_norm": (c_int, [c_void_p, c_void_p, c_int64, c_float, c_void_p, c_float, c_void_p, c_void_p, c_int64, c_int,
                               c_int, c_float, c_int, c_void_p]),
-    "dz_residual_norm": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int64,
-                                 c_int, c_int, c_float, c_int, c_void_p]),
+    "dz_residual_norm": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                 c_float, c_void_p, c_int64, c_int, c_int, c_float, c_int, c_void_p]),
+    "dz_act": (c_int, [c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "dz_gated_act": (c_int, [c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "dz_qk_norm": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
                            c_void_p, c_int, c_int, c_void_p]),
@@ -145,6 +181,20 @@ _SIGNATURES = {
     "dz_mlstm_chunk_supported": (c_int, [c_int, c_int, c_int]),
     "dz_mlstm_workspace_bytes": (c_size_t, [c_int, c_int]),
     "dz_mlstm": (c_int, [POINTER(MlstmArgs), c_void_p]),
+    "dz_latent_rows": (c_int, [POINTER(LatentRowsArgs), c_void_p]),
+    "dz_latent_gather": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
+                                 c_void_p]),
+    "dz_latent_attention_ctas": (c_int, [c_int, c_int, c_int, c_int, c_int]),
+    "dz_latent_attention_workspace_bytes": (c_size_t, [c_int, c_int, c_int, c_int]),
+    "dz_latent_attention": (c_int, [POINTER(LatentAttentionArgs), c_void_p]),
+    "dz_lightning_chunk_supported": (c_int, [c_int, c_int, c_int]),
+    "dz_lightning_workspace_bytes": (c_size_t, [c_int, c_int, c_int, c_int, c_int]),
+    "dz_lightning": (c_int, [POINTER(LightningArgs), c_void_p]),
+    "dz_moe_route": (c_int, [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
+    "dz_moe_sort": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "dz_moe_gather": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p]),
+    "dz_moe_gemm": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                            c_int, c_void_p, c_void_p]),
     "dz_slot_upload": (c_int, [c_void_p, c_void_p, c_size_t, c_int, c_void_p]),
     "dz_slot_reset": (c_int, [c_void_p, c_size_t, c_void_p]),
     "dz_stream_fence": (c_int, [c_void_p]),

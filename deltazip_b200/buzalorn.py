@@ -18,10 +18,9 @@ import torch
 import torch.nn as nn
 
 from . import ops
-from .cache import AttnMeta, PagedKVCache, RecurrentStateCache
-from .loader import copy_weights
+from .cache import AttnMeta, PagedKVCache
+from .decoder import DecoderLayer, LayeredDecoder
 from .mixers import GatedMLP, Mlstm, MlstmSpec, WindowAttention, WindowAttentionSpec
-from .parallel_state import get_tensor_model_parallel_world_size
 
 NORM_OFFSET = 1.0                       # norms multiply by (1 + w)
 DEFAULT_BIAS_ROWS = 32                  # of a model made without a checkpoint
@@ -72,65 +71,31 @@ class BuzalornConfig:
         return out + [(i, None) for i in range(self.loop_stop, len(self.layers))]
 
 
-class BuzalornLayer(nn.Module):
-    def __init__(self, spec: LayerSpec, cfg: BuzalornConfig, bias_rows: int, device, dtype):
-        super().__init__()
-        if isinstance(spec.mixer, MlstmSpec):
-            self.mixer = Mlstm(spec.mixer, cfg.width, cfg.eps, device, dtype)
-        else:
-            self.mixer = WindowAttention(spec.mixer, cfg.width, bias_rows, cfg.eps, device, dtype)
-        norm = lambda: nn.Parameter(torch.zeros(cfg.width, dtype=torch.float32, device=device), requires_grad=False)
-        self.norm1 = norm()
-        self.mlp = self.norm2 = None
-        if spec.ff is not None:
-            self.norm2 = norm()
-            self.mlp = GatedMLP(cfg.width, spec.ff, "gelu_tanh", device, dtype)
-
-
-class BuzalornForCausalLM(nn.Module):
+class BuzalornForCausalLM(LayeredDecoder):
     supported_delta_modules = ["qkv_proj", "qkvg_proj", "o_proj", "gate_up_proj", "down_proj"]
     packed_modules_mapping = {"gate_up_proj": ["gate_proj", "up_proj"]}
-    supports_portions = True            # a prompt may be continued from the cache and state
 
     def __init__(self, cfg: BuzalornConfig, device="cuda", seed: int = 0, dtype=torch.bfloat16,
                  bias_rows: Union[int, Dict[int, int]] = DEFAULT_BIAS_ROWS):
         """`bias_rows`: rows of the attention layers' distance tables (per layer index when a dict); it
         is a tensor's shape, not a configuration value."""
-        super().__init__()
-        if get_tensor_model_parallel_world_size() != 1:
-            raise ValueError("this model runs on one rank")
-        # 16-bit GEMMs accumulate in 32 bits throughout, 32-bit ones use no reduced-precision mode
-        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
-        torch.backends.cuda.matmul.allow_fp16_reduced_precision_reduction = False
-        if dtype == torch.float32:
-            torch.backends.cuda.matmul.allow_tf32 = False
-        self.cfg, self.dtype = cfg, dtype
-        gen = torch.Generator(device=device).manual_seed(seed)
-        par = lambda *shape, std, dt=dtype: nn.Parameter(
-            torch.empty(shape, dtype=dt, device=device).normal_(0, std, generator=gen), requires_grad=False)
-        f32 = torch.float32
-        self.embed_tokens = par(cfg.vocab_size, cfg.width, std=1.0)
-        self.embed_norm, self.norm = par(cfg.width, std=0.0, dt=f32), par(cfg.width, std=0.0, dt=f32)
-        self.loop_in = par(cfg.width, 2 * cfg.width, std=(2 * cfg.width) ** -0.5)
-        self.loop_step = par(cfg.loop_times, cfg.width, std=0.1, dt=f32)
-        rows = (lambda i: bias_rows[i]) if isinstance(bias_rows, dict) else (lambda i: bias_rows)
-        self.layers = nn.ModuleList([
-            BuzalornLayer(spec, cfg, rows(i) if isinstance(spec.mixer, WindowAttentionSpec) else 0, device, dtype)
-            for i, spec in enumerate(cfg.layers)])
-        # cache runs: the n-th key/value pool or state pool belongs to the n-th such layer run
-        self.plan, count = [], {"kv": 0, "state": 0}
-        self._kv_shapes, self._state_shapes = [], []
-        for i, first_of_pass in cfg.runs():
-            s, kind = cfg.layers[i].mixer, self.layers[i].mixer.kind
-            self.plan.append((self.layers[i], count[kind], first_of_pass))
-            count[kind] += 1
-            if kind == "kv":
-                self._kv_shapes.append((s.kv_heads, s.dim, s.vdim))
+        super().__init__(cfg, device, seed, dtype)
+        f32, w = torch.float32, cfg.width
+        self.embed_tokens = self._random(cfg.vocab_size, w, std=1.0)
+        self.embed_norm, self.norm = self._random(w, std=0.0, dtype=f32), self._random(w, std=0.0, dtype=f32)
+        self.loop_in = self._random(w, 2 * w, std=(2 * w) ** -0.5)
+        self.loop_step = self._random(cfg.loop_times, w, std=0.1, dtype=f32)
+        self.layers = nn.ModuleList()
+        for i, spec in enumerate(cfg.layers):
+            if isinstance(spec.mixer, MlstmSpec):
+                mixer = Mlstm(spec.mixer, w, cfg.eps, device, dtype)
             else:
-                self._state_shapes.append((s.heads, s.dim, s.vdim))
-        windows = [x.mixer.window for x in cfg.layers if isinstance(x.mixer, WindowAttentionSpec)]
-        self.window = max(windows, default=0)
-        self.kv_heads = max([h for h, _, _ in self._kv_shapes], default=1)
+                rows = bias_rows[i] if isinstance(bias_rows, dict) else bias_rows
+                mixer = WindowAttention(spec.mixer, w, rows, cfg.eps, device, dtype)
+            mlp = GatedMLP(w, spec.ff, "gelu_tanh", device, dtype) if spec.ff is not None else None
+            self.layers.append(DecoderLayer(mixer, mlp, w, 0.0, device))
+        runs = self.plan_cache([i for i, _ in cfg.runs()])
+        self.plan = [(self.layers[i], run, first_of_pass) for (i, first_of_pass), run in zip(cfg.runs(), runs)]
         self.finalize()
 
     # -- weights -----------------------------------------------------------------------
@@ -144,28 +109,9 @@ class BuzalornForCausalLM(nn.Module):
         model.load_weights(tensors)
         return model
 
-    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
-        want = {"embed": [self.embed_tokens], "embed.norm": [self.embed_norm], "final.norm": [self.norm],
-                "loop.in": [self.loop_in], "loop.step": [self.loop_step]}
-        for i, layer in enumerate(self.layers):
-            want[f"l{i}.norm1"] = [layer.norm1]
-            want.update({f"l{i}.mix.{k}": [v] for k, v in layer.mixer.weight_views().items()})
-            if layer.mlp is not None:
-                want[f"l{i}.norm2"] = [layer.norm2]
-                want.update({f"l{i}.mlp.{k}": [v] for k, v in layer.mlp.weight_views().items()})
-        copy_weights(want, tensors)
-        self.finalize()
-
-    def finalize(self) -> None:
-        for layer in self.layers:
-            layer.mixer.prepare()
-
-    # -- cache -------------------------------------------------------------------------
-    def make_cache(self, num_blocks: int, block_size: int, max_seqs: int) -> PagedKVCache:
-        device = self.embed_tokens.device
-        state = RecurrentStateCache(self._state_shapes, max_seqs, device) if self._state_shapes else None
-        return PagedKVCache(len(self._kv_shapes), num_blocks, self.kv_heads, block_size, self.dtype, device,
-                            layer_shapes=self._kv_shapes, window=self.window, state=state)
+    def top_weights(self) -> Dict[str, torch.Tensor]:
+        return {"embed": self.embed_tokens, "embed.norm": self.embed_norm, "final.norm": self.norm,
+                "loop.in": self.loop_in, "loop.step": self.loop_step}
 
     # -- forward -----------------------------------------------------------------------
     def forward(self, tokens: torch.Tensor, positions: torch.Tensor, cache: PagedKVCache, meta: AttnMeta,
@@ -197,6 +143,3 @@ class BuzalornForCausalLM(nn.Module):
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         """float32 logits; the output matrix is the embedding table."""
         return ops.matmul_f32(hidden, self.embed_tokens) * self.cfg.logit_scale
-
-    def greedy_tokens(self, hidden: torch.Tensor) -> torch.Tensor:
-        return self.logits(hidden).argmax(dim=-1)

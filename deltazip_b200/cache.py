@@ -4,22 +4,25 @@ block manager + cache engine, serving/vllm/core/block_manager.py,
 serving/vllm/worker/cache_engine.py, reduced to what a single process needs)."""
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import List, Optional, Sequence, Tuple
 
 import torch
 
 
 class RecurrentStateCache:
-    """Per recurrent layer run the 32-bit pools S [slots, heads, dim, vdim], n [slots, heads, dim] and
-    m [slots, heads]; a sequence owns one slot number, the same in every pool.  Slots are handed out
-    as they are: a sequence without context starts from zero without reading its slot."""
+    """Per recurrent layer run the 32-bit pools S [slots, heads, dim, vdim] and, where the run normalises
+    (`normalised`, default: all do), n [slots, heads, dim] and m [slots, heads]; a sequence owns one
+    slot number, the same in every pool.  Slots are handed out as they are: a sequence without context
+    starts from zero without reading its slot."""
 
-    def __init__(self, shapes: Sequence[Tuple[int, int, int]], slots: int, device="cuda"):
+    def __init__(self, shapes: Sequence[Tuple[int, int, int]], slots: int, device="cuda",
+                 normalised: Optional[Sequence[bool]] = None):
         f32 = dict(dtype=torch.float32, device=device)
+        with_n = [True] * len(shapes) if normalised is None else list(normalised)
         self.S = [torch.zeros((slots, h, d, v), **f32) for h, d, v in shapes]
-        self.n = [torch.zeros((slots, h, d), **f32) for h, d, _ in shapes]
-        self.m = [torch.zeros((slots, h), **f32) for h, _, _ in shapes]
+        self.n = [torch.zeros((slots, h, d), **f32) if w else None for (h, d, _), w in zip(shapes, with_n)]
+        self.m = [torch.zeros((slots, h), **f32) if w else None for (h, _, _), w in zip(shapes, with_n)]
         self.free: List[int] = list(range(slots - 1, -1, -1))
 
     def allocate(self) -> int:
@@ -34,7 +37,8 @@ class RecurrentStateCache:
 class PagedKVCache:
     """Per-layer K and V pools of `num_blocks` blocks of `block_size` tokens, [slots, kv_heads,
     head size] each, with a free list.  `layer_shapes` gives (kv_heads, key size, value size) per
-    layer run where layers differ (default: `num_layers` times (kv_heads, 128, 128)).
+    layer run where layers differ (default: `num_layers` times (kv_heads, 128, 128)); a run that caches
+    one row per token for all heads has one key head and value size 0.
 
     `window`: the largest number of tokens any layer looks back (itself included).  A sequence then
     owns at most ceil(window / block_size) blocks and uses them as a ring: token position t lives in
@@ -105,8 +109,9 @@ class AttnMeta:
     Prompt portions: `prompt_lens`, the row count of each sequence.
 
     Models that continue prompts from a cache also read `q_starts` [B + 1] int32 (first row of every
-    sequence), `ctx_lens` [B] int32 (tokens before the first row) and, with recurrent layers,
-    `state_slots` [B] int32."""
+    sequence), `ctx_lens` [B] int32 (tokens before the first row; `host_ctx_lens` the same as numbers, for
+    prompt portions) and, with recurrent layers, `state_slots` [B] int32.  `shared` keeps what the layers
+    of one pass derive from all this."""
     slot_mapping: Optional[torch.Tensor] = None          # int64 [M] cache slot per token, -1 = none
     block_tables: Optional[torch.Tensor] = None
     seq_lens: Optional[torch.Tensor] = None
@@ -115,6 +120,9 @@ class AttnMeta:
     q_starts: Optional[torch.Tensor] = None
     ctx_lens: Optional[torch.Tensor] = None
     state_slots: Optional[torch.Tensor] = None
+    host_ctx_lens: Optional[List[int]] = None
+    positions: Optional[torch.Tensor] = None             # int64 [M], set by models whose mixers read them
+    shared: dict = field(default_factory=dict)
 
     @property
     def decode(self) -> bool:

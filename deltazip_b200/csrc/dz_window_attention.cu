@@ -13,6 +13,10 @@
 // never has to hold more than a window.  A decoded token is appended before attention, inside the
 // query / key norm.
 //
+// Keys and values may also lie in rows of their own (`kv`, all positions of a sequence from
+// kv_starts[sequence] on), and a row may have a sink: one more score in the softmax's denominator,
+// not scaled, without a key or a value.
+//
 // Scores, softmax weights and sums are 32-bit.  In the tensor-core kernel a weight enters its
 // product with v as a hi + lo pair of 16-bit numbers.
 #include "dz_window_attention.cuh"
@@ -129,7 +133,9 @@ attention_any_kernel(AttnParams p, int num_seqs) {
   const int seq = s_seq, q0 = p.q_starts[seq], ctx = p.ctx_lens[seq], pos = ctx + row - q0;
   const int* table = p.block_tables + (size_t)seq * p.ring_blocks;
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-  float m = -INFINITY, l = 0.f, acc[kAnyMaxV];
+  const KeyRows kr(p, seq, q0, ctx);
+  const T* kv = (const T*)p.kv;
+  float m = p.sink ? p.sink[head] : -INFINITY, l = p.sink ? 1.f : 0.f, acc[kAnyMaxV];
 #pragma unroll
   for (int c = 0; c < kAnyMaxV; ++c) acc[c] = 0.f;
   for (int t0 = lo; t0 <= pos; t0 += kAnyThreads) {
@@ -137,8 +143,8 @@ attention_any_kernel(AttnParams p, int num_seqs) {
     for (int k = warp; k < n; k += kAnyThreads / 32) {
       const int t = t0 + k;
       const T* kp;
-      if (t >= ctx) {
-        kp = qkv + (size_t)(q0 + t - ctx) * p.row_stride + p.k_off + (size_t)kvh * p.dim;
+      if (t >= kr.first) {
+        kp = kv + (size_t)(kr.row + t - kr.first) * p.kv_stride + p.k_off + (size_t)kvh * p.dim;
       } else {
         kp = (const T*)p.k_cache + (ring_slot(p, table, t) * p.kv_heads + kvh) * p.dim;
       }
@@ -149,8 +155,8 @@ attention_any_kernel(AttnParams p, int num_seqs) {
         s = s * p.scale;
         if (p.bias) s += p.bias[(size_t)head * p.bias_len + min(pos - t, p.bias_len - 1)];
         s_w[k] = s;
-        s_v[k] = t >= ctx ? (size_t)(q0 + t - ctx) * p.row_stride + p.v_off + (size_t)kvh * p.vdim
-                          : (ring_slot(p, table, t) * p.kv_heads + kvh) * p.vdim;
+        s_v[k] = t >= kr.first ? (size_t)(kr.row + t - kr.first) * p.kv_stride + p.v_off + (size_t)kvh * p.vdim
+                               : (ring_slot(p, table, t) * p.kv_heads + kvh) * p.v_row;
       }
     }
     __syncthreads();
@@ -170,7 +176,7 @@ attention_any_kernel(AttnParams p, int num_seqs) {
       if (d < p.vdim) {
         float a = acc[v] * c;
         for (int k = 0; k < n; ++k)
-          a += s_w[k] * Cvt<T>::one((t0 + k >= ctx ? qkv : (const T*)p.v_cache)[s_v[k] + d]);
+          a += s_w[k] * Cvt<T>::one((t0 + k >= kr.first ? kv : (const T*)p.v_cache)[s_v[k] + d]);
         acc[v] = a;
       }
     }
@@ -257,8 +263,8 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
       const int d = (c * 16 + hl) * 8;
       va[c] = vb[c] = make_uint4(0, 0, 0, 0);
       if (d < p.vdim) {
-        va[c] = *reinterpret_cast<const uint4*>(vc + ra * p.vdim + d);
-        vb[c] = *reinterpret_cast<const uint4*>(vc + rb * p.vdim + d);
+        va[c] = *reinterpret_cast<const uint4*>(vc + ra * p.v_row + d);
+        vb[c] = *reinterpret_cast<const uint4*>(vc + rb * p.v_row + d);
       }
     }
     float pa[G], pb[G];
@@ -354,6 +360,11 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
     }
     const int head = kvh * ratio + g0 + g;
     if (splits == 1) {
+      if (p.sink) {
+        const float sk = p.sink[head], top = fmaxf(mm, sk), c = __expf(mm - top);
+        a *= c;
+        ll = ll * c + __expf(sk - top);
+      }
       ((T*)p.out)[((size_t)seq * p.heads + head) * p.vdim + d] = Cvt<T>::from(a / ll);
     } else {
       float* pp = partial + (((size_t)seq * p.heads + head) * splits + split) * (p.vdim + 2);
@@ -377,7 +388,8 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
     const float* pp = partial + ((size_t)seq * p.heads + head) * splits * w;
     float mm = -INFINITY;
     for (int s = 0; s < splits; ++s) mm = fmaxf(mm, __ldcg(pp + s * w + p.vdim));
-    float ll = 0.f, a = 0.f;
+    if (p.sink) mm = fmaxf(mm, p.sink[head]);
+    float ll = p.sink ? __expf(p.sink[head] - mm) : 0.f, a = 0.f;
     for (int s = 0; s < splits; ++s) {
       const float ms = __ldcg(pp + s * w + p.vdim);
       const float c = ms == -INFINITY ? 0.f : __expf(ms - mm);
@@ -417,6 +429,8 @@ window_prefill_kernel(AttnParams p, int dimp) {
   const int vcols = min(DVP, p.vdim - v0);
   const int* table = p.block_tables + (size_t)seq * p.ring_blocks;
   const T* qkv = (const T*)p.qkv;
+  const T* kv = (const T*)p.kv;
+  const KeyRows kr(p, seq, q0, ctx);
   const int blen = p.bias ? p.bias_len : 0;
   const bool bias_in_smem = blen <= kBiasSmem;
   const float* gbias = p.bias ? p.bias + (size_t)head * p.bias_len : nullptr;
@@ -443,14 +457,14 @@ window_prefill_kernel(AttnParams p, int dimp) {
     const int t = t0 + r;
     const bool ok = t < end;
     const T *ks, *vs;
-    if (!ok || t >= ctx) {
-      const T* row = qkv + (size_t)(q0 + (ok ? t - ctx : 0)) * p.row_stride;
+    if (!ok || t >= kr.first) {
+      const T* row = kv + (size_t)(ok ? kr.row + t - kr.first : 0) * p.kv_stride;
       ks = row + p.k_off + (size_t)kvh * p.dim;
       vs = row + p.v_off + (size_t)kvh * p.vdim;
     } else {
       const size_t s = ring_slot(p, table, t) * p.kv_heads + kvh;
       ks = (const T*)p.k_cache + s * p.dim;
-      vs = (const T*)p.v_cache + s * p.vdim;
+      vs = (const T*)p.v_cache + s * p.v_row;
     }
     T* dk = sk + (buf * kBN + r) * ldk;
     T* dv = sv + (buf * kBN + r) * ldv;
@@ -459,6 +473,10 @@ window_prefill_kernel(AttnParams p, int dimp) {
   };
 
   float o[NT][4], mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+  if (p.sink) {
+    mrow[0] = mrow[1] = p.sink[head] * kLog2e;
+    lrow[0] = lrow[1] = (lane & 3) == 0 ? 1.f : 0.f;
+  }
 #pragma unroll
   for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -633,10 +651,19 @@ size_t ticket_bytes(int num_seqs, int heads, int kv_heads) {
 // The 16-byte copies of the fast kernels need 8-element rows everywhere.
 bool fast_shapes(const AttnParams& p, int dtype) {
   return dtype != DZ_DTYPE_F32 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.row_stride % 8 == 0 && p.k_off % 8 == 0 &&
-         p.v_off % 8 == 0 && aligned16(p.qkv) && aligned16(p.out) && aligned16(p.k_cache) && aligned16(p.v_cache);
+         p.v_off % 8 == 0 && p.v_row % 8 == 0 && p.kv_stride % 8 == 0 && aligned16(p.qkv) && aligned16(p.out) &&
+         aligned16(p.k_cache) && aligned16(p.v_cache) && aligned16(p.kv);
 }
 
 }  // namespace
+
+int launch_attention_any(const AttnParams& p, int num_seqs, int dtype, cudaStream_t st) {
+  if (p.vdim > kAnyMaxV * kAnyThreads || p.dim > 8192 || p.heads > 65535) return DZ_ERR_SHAPE;
+  DZ_DISPATCH(dtype, DZ_CUDA_OK(launch_ex(attention_any_kernel<T>, dim3(p.rows, p.heads), dim3(kAnyThreads),
+                                          (size_t)p.dim * 4, 1, st, p, num_seqs)));
+  return DZ_OK;
+}
+
 }  // namespace dz
 
 using namespace dz;
@@ -678,29 +705,28 @@ size_t dz_window_attention_workspace_bytes(int num_seqs, int heads, int kv_heads
 }
 
 int dz_window_attention(const dz_window_attention_args* a, void* stream) {
-  if (!a || !a->qkv || !a->out || !a->k_cache || !a->v_cache || !a->block_tables || !a->q_starts || !a->ctx_lens)
+  const bool own = a && a->kv;                     // keys and values in rows of their own
+  if (!a || !a->qkv || !a->out || !a->q_starts || !a->ctx_lens) return DZ_ERR_INVALID_ARG;
+  if (own ? (!a->kv_starts || a->kv_rows <= 0 || a->decode) : (!a->k_cache || !a->v_cache || !a->block_tables))
     return DZ_ERR_INVALID_ARG;
   if (a->num_seqs < 0 || a->rows < 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 ||
-      a->vdim <= 0 || a->ring_blocks <= 0 || a->block_size <= 0 || a->splits < 1 || a->splits > 64 ||
+      a->vdim <= 0 || (!own && (a->ring_blocks <= 0 || a->block_size <= 0)) || a->splits < 1 || a->splits > 64 ||
       (a->bias && a->bias_len <= 0) || !is_float_dtype(a->dtype))
     return DZ_ERR_INVALID_ARG;
-  if (a->k_off < 0 || a->v_off < 0 || a->row_stride < (int64_t)a->v_off + (int64_t)a->kv_heads * a->vdim ||
-      a->row_stride < (int64_t)a->k_off + (int64_t)a->kv_heads * a->dim ||
+  const int64_t kv_stride = own ? a->kv_stride : a->row_stride;
+  if (a->k_off < 0 || a->v_off < 0 || kv_stride < (int64_t)a->v_off + (int64_t)a->kv_heads * a->vdim ||
+      kv_stride < (int64_t)a->k_off + (int64_t)a->kv_heads * a->dim ||
       a->row_stride < (int64_t)a->heads * a->dim)
     return DZ_ERR_INVALID_ARG;
   if (a->num_seqs == 0 || a->rows == 0) return DZ_OK;
   if (a->num_seqs > 65535 || (a->decode && a->rows != a->num_seqs)) return DZ_ERR_INVALID_ARG;
-  AttnParams p = {a->qkv, a->row_stride, a->k_off, a->v_off, a->out, a->k_cache, a->v_cache, a->block_tables,
+  AttnParams p = {a->qkv, a->row_stride, a->k_off, a->v_off, a->out, a->k_cache, a->v_cache, a->vdim, a->block_tables,
                   a->ring_blocks, a->block_size, a->q_starts, a->ctx_lens, a->heads, a->kv_heads, a->dim, a->vdim,
-                  a->scale, a->window, a->bias, a->bias_len, a->rows, nullptr};
+                  a->scale, a->window, a->bias, a->bias_len, a->rows, a->sink, own ? kKeysRows : kKeysSplit,
+                  own ? a->kv : a->qkv, kv_stride, a->kv_starts, own ? a->kv_rows : a->rows, nullptr};
   if (a->workspace && a->workspace_bytes >= kAttnStatusBytes) p.status = (int*)a->workspace;
   cudaStream_t st = (cudaStream_t)stream;
-  if (!fast_shapes(p, a->dtype)) {
-    if (a->vdim > kAnyMaxV * kAnyThreads || a->dim > 8192 || a->heads > 65535) return DZ_ERR_SHAPE;
-    DZ_DISPATCH(a->dtype, DZ_CUDA_OK(launch_ex(attention_any_kernel<T>, dim3(a->rows, a->heads), dim3(kAnyThreads),
-                                               (size_t)a->dim * 4, 1, st, p, a->num_seqs)));
-    return DZ_OK;
-  }
+  if (!fast_shapes(p, a->dtype)) return launch_attention_any(p, a->num_seqs, a->dtype, st);
   if (a->decode && a->dim <= 256 && a->vdim <= 256) {
     float* partial = nullptr;
     int* tickets = nullptr;
@@ -724,12 +750,8 @@ int dz_window_attention(const dz_window_attention_args* a, void* stream) {
   const int dvp = a->vdim <= 64 ? 64 : a->vdim <= 96 ? 96 : a->vdim <= 128 ? 128 : a->vdim <= 192 ? 192 : 256;
   const size_t bias_bytes = a->bias && a->bias_len <= kBiasSmem ? (size_t)a->bias_len * 4 : 0;
   const size_t smem = ((size_t)(kBM + 2 * kBN) * (dimp + 8) + (size_t)2 * kBN * (dvp + 8)) * 2 + bias_bytes;
-  if (smem > kMaxDynSmem || (int64_t)a->heads * ((a->vdim + dvp - 1) / dvp) > 65535) {
-    if (a->vdim > kAnyMaxV * kAnyThreads || a->dim > 8192 || a->heads > 65535) return DZ_ERR_SHAPE;
-    DZ_DISPATCH16(a->dtype, DZ_CUDA_OK(launch_ex(attention_any_kernel<T>, dim3(a->rows, a->heads), dim3(kAnyThreads),
-                                                 (size_t)a->dim * 4, 1, st, p, a->num_seqs)));
-    return DZ_OK;
-  }
+  if (smem > kMaxDynSmem || (int64_t)a->heads * ((a->vdim + dvp - 1) / dvp) > 65535)
+    return launch_attention_any(p, a->num_seqs, a->dtype, st);
   DZ_DISPATCH16(a->dtype, switch (dvp) {
     case 64: return run_prefill<T, 64>(p, a->num_seqs, max_q, dimp, smem, st);
     case 96: return run_prefill<T, 96>(p, a->num_seqs, max_q, dimp, smem, st);

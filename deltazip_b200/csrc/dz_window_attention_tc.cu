@@ -4,7 +4,7 @@
 // TMEM lane) and walks the keys in tiles of 64 that both read.  Roles of its twelve warps:
 //   0-3, 4-7  softmax of query tile 0 / 1: a thread owns a row -- scores from TMEM into registers,
 //             scale + bias + mask, running maximum, exponentials, weights back to TMEM
-//   8-9       copies into 128-byte-swizzled shared memory, four stages: TMA where a tile lies in the
+//   8-9       copies into 128-byte-swizzled shared memory, three or four stages: TMA where a tile lies in the
 //             projection rows, 16-byte asynchronous copies where it comes from the cache ring or ends
 //             with the sequence
 //   10, 11    MMA issue for query tile 0 / 1: S = Q K^T (both operands in shared memory), O += P V
@@ -27,7 +27,8 @@
 namespace dz {
 namespace {
 
-constexpr int kTileM = 128, kTileKeys = 64, kStages = 4;
+constexpr int kTileM = 128, kTileKeys = 64, kMaxStages = 4;
+constexpr int kMaxDim = 192;                            // then the shared memory holds three stages of keys
 constexpr int kThreadsTc = 384, kCopyThreads = 64;
 constexpr int kSlabQ = kTileM * 128, kSlab = kTileKeys * 128;   // rows of 64 16-bit elements
 constexpr int kBiasTc = 4096;
@@ -130,9 +131,10 @@ __device__ __forceinline__ void bar_wait(uint64_t* bar, uint32_t parity, volatil
   mbar_wait_slow(smem_u32(bar), parity, abort_flag, status);
 }
 
-template <typename T>
+template <typename T, int kStages>
 __global__ void __launch_bounds__(kThreadsTc, 1)
-window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnParams p) {
+window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
+                         const AttnParams p) {
   constexpr int DT = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
   extern __shared__ uint8_t smem_dyn[];
   __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2][2], b_p[2][2], b_pv[2], b_o[2], b_q;
@@ -153,7 +155,9 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
   float* s_bias = reinterpret_cast<float*>(smem_dyn + (s_v + kStages * vs * kSlab - smem_u32(smem_dyn)));
   volatile int* abort_flag = &s_abort;
   const T* qkv = (const T*)p.qkv;
+  const T* kv = (const T*)p.kv;
   const int* table = p.block_tables + (size_t)seq * p.ring_blocks;
+  const KeyRows kr(p, seq, q0, ctx);
 
   // key tiles: all of the CTA's, and of those the range [ta, tb) with keys a query tile may see
   const int first = p.window > 0 ? max(0, ctx + m0 - p.window + 1) : 0;
@@ -257,7 +261,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
         mbar_expect_tx(bar, 2 * ks * kSlabQ);
         for (int i = 0; i < 2 * ks; ++i)                          // two boxes of 64 rows fill a slab
           for (int half = 0; half < 2; ++half)
-            tma_load_2d(s_q + i * kSlabQ + half * (kSlabQ / 2), &map, head * p.dim + (i % ks) * 64,
+            tma_load_2d(s_q + i * kSlabQ + half * (kSlabQ / 2), &map_q, head * p.dim + (i % ks) * 64,
                         q0 + m0 + (i / ks) * kTileM + half * 64, bar);
       } else {
         mbar_arrive(bar);
@@ -267,12 +271,12 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
       const int st = j % kStages, key0 = first + j * kTileKeys;
       bar_wait(&b_empty[st], ((j / kStages) & 1) ^ 1, abort_flag, p.status);
       const uint32_t dk = s_k + st * ks * kSlab, dv = s_v + st * vs * kSlab, full = smem_u32(&b_full[st]);
-      if (key0 >= ctx && key0 + kTileKeys <= end) {
+      if (key0 >= kr.first && key0 + kTileKeys <= end) {
         if (t == 0) {
-          const int row = q0 + key0 - ctx;
+          const int row = kr.row + key0 - kr.first;
           mbar_expect_tx(full, (ks + vs) * kSlab);
-          for (int i = 0; i < ks; ++i) tma_load_2d(dk + i * kSlab, &map, p.k_off + kvh * p.dim + i * 64, row, full);
-          for (int i = 0; i < vs; ++i) tma_load_2d(dv + i * kSlab, &map, p.v_off + kvh * p.vdim + v0 + i * 64, row, full);
+          for (int i = 0; i < ks; ++i) tma_load_2d(dk + i * kSlab, &map_kv, p.k_off + kvh * p.dim + i * 64, row, full);
+          for (int i = 0; i < vs; ++i) tma_load_2d(dv + i * kSlab, &map_kv, p.v_off + kvh * p.vdim + v0 + i * 64, row, full);
         } else {
           mbar_arrive(full);
         }
@@ -283,18 +287,17 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
         const int key = key0 + r;
         const bool ok = key < end;
         const T *kp, *vp;
-        if (!ok || key >= ctx) {
-          const T* row = qkv + (size_t)(q0 + (ok ? key - ctx : 0)) * p.row_stride;
+        if (!ok || key >= kr.first) {
+          const T* row = kv + (size_t)(ok ? kr.row + key - kr.first : 0) * p.kv_stride;
           kp = row + p.k_off + (size_t)kvh * p.dim;
           vp = row + p.v_off + (size_t)kvh * p.vdim;
         } else {
           const size_t slot = ring_slot(p, table, key) * p.kv_heads + kvh;
           kp = (const T*)p.k_cache + slot * p.dim;
-          vp = (const T*)p.v_cache + slot * p.vdim;
+          vp = (const T*)p.v_cache + slot * p.v_row;
         }
-        const uint32_t at = swizzled(r, c, kSlab);
-        if (c < p.dim / 8) cp_async16_u32(dk + at, kp + c * 8, ok);
-        if (c < vcols / 8) cp_async16_u32(dv + at, vp + v0 + c * 8, ok);
+        for (int e = c; e < p.dim / 8; e += 16) cp_async16_u32(dk + swizzled(r, e, kSlab), kp + e * 8, ok);
+        if (c < vcols / 8) cp_async16_u32(dv + swizzled(r, c, kSlab), vp + v0 + c * 8, ok);
       }
       cp_async_commit();
       cp_async_wait<0>();
@@ -304,8 +307,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
   } else {
     // ---- softmax ----
     if (!q_tma) {
-      const int c = tid & 15;
-      if (c < p.dim / 8) {
+      for (int c = tid & 15; c < p.dim / 8; c += 16) {
         for (int i = tid >> 4; i < 2 * kTileM; i += 16) {
           const bool ok = m0 + i < qn;
           const T* src = qkv + (size_t)(q0 + (ok ? m0 + i : 0)) * p.row_stride + (size_t)head * p.dim + c * 8;
@@ -327,7 +329,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t t_o = tmem + 256 + g * 128 + lane_addr;
     const float scale2 = p.scale * kLog2e, far_bias = s_bias[kBiasPad + blen - 1];
-    float m = -INFINITY, l = 0.f;
+    float m = p.sink ? p.sink[head] * kLog2e : -INFINITY, l = p.sink ? 1.f : 0.f;
     for (int j = ta; j < tb; ++j) {
       const int n = j - ta, buf = n & 1;
       const uint32_t t_s = tmem + g * 128 + buf * 64 + lane_addr;
@@ -445,8 +447,10 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, const AttnPara
   }
 }
 
+int tc_stages(const AttnParams& p) { return p.dim <= 128 ? kMaxStages : kMaxStages - 1; }
+
 size_t tc_smem(const AttnParams& p) {
-  const int ks = (p.dim + 63) / 64, vs = (std::min(128, p.vdim) + 63) / 64;
+  const int kStages = tc_stages(p), ks = (p.dim + 63) / 64, vs = (std::min(128, p.vdim) + 63) / 64;
   const int blen = p.bias ? p.bias_len : 1;
   return (size_t)2 * ks * kSlabQ + (size_t)kStages * (ks + vs) * kSlab + (size_t)(blen + 2 * kBiasPad) * 4 + 1024;
 }
@@ -454,20 +458,23 @@ size_t tc_smem(const AttnParams& p) {
 template <typename T>
 int run(const AttnParams& p, int num_seqs, int max_q, cudaStream_t st) {
   const size_t smem = tc_smem(p);
-  CUtensorMap map;
-  const int rc = make_map(&map, p.qkv, p.rows, (int)p.row_stride, kTileKeys, std::is_same<T, __nv_bfloat16>::value);
+  constexpr int kDt = std::is_same<T, __nv_bfloat16>::value;
+  CUtensorMap map_q, map_kv;
+  int rc = make_map(&map_q, p.qkv, p.rows, (int)p.row_stride, kTileKeys, kDt);
+  if (!rc) rc = make_map(&map_kv, p.kv, p.kv_rows, (int)p.kv_stride, kTileKeys, kDt);
   if (rc) return rc;
   const dim3 grid((max_q + 2 * kTileM - 1) / (2 * kTileM), p.heads * ((p.vdim + 127) / 128), num_seqs);
-  DZ_CUDA_OK(allow_smem(window_prefill_tc_kernel<T>, smem));
-  DZ_CUDA_OK(launch_ex(window_prefill_tc_kernel<T>, grid, dim3(kThreadsTc), smem, 1, st, map, p));
+  auto kern = tc_stages(p) == kMaxStages ? window_prefill_tc_kernel<T, kMaxStages> : window_prefill_tc_kernel<T, kMaxStages - 1>;
+  DZ_CUDA_OK(allow_smem(kern, smem));
+  DZ_CUDA_OK(launch_ex(kern, grid, dim3(kThreadsTc), smem, 1, st, map_q, map_kv, p));
   return DZ_OK;
 }
 
 }  // namespace
 
 bool window_prefill_tc_supported(const AttnParams& p, int dtype) {
-  return (dtype == DZ_DTYPE_F16 || dtype == DZ_DTYPE_BF16) && p.dim <= 128 && p.dim % 8 == 0 &&
-         p.row_stride < (1ll << 31) && p.vdim % 8 == 0 &&
+  return (dtype == DZ_DTYPE_F16 || dtype == DZ_DTYPE_BF16) && p.dim <= kMaxDim && p.dim % 8 == 0 &&
+         p.row_stride < (1ll << 31) && p.kv_stride < (1ll << 31) && tc_smem(p) <= kMaxDynSmem && p.vdim % 8 == 0 &&
          (!p.bias || p.bias_len <= kBiasTc) && p.heads * ((p.vdim + 127) / 128) <= 65535;
 }
 

@@ -254,7 +254,7 @@ class DecodeEngine:
             seq_lens=self._int32([s.length + n for s, n in zip(seqs, counts)]),
             prompt_lens=None if decode else counts,
             q_starts=self._int32(starts), ctx_lens=self._int32([s.length for s in seqs]),
-            state_slots=self._state_slots(seqs))
+            state_slots=self._state_slots(seqs), host_ctx_lens=[s.length for s in seqs])
         toks = torch.tensor([t for _, ts in work for t in ts], dtype=torch.int64).to(dev)
         pos = torch.tensor([s.length + i for s, n in zip(seqs, counts) for i in range(n)], dtype=torch.int64).to(dev)
         self._set_mapping(seqs, counts)

@@ -3,13 +3,15 @@ attention of llama.py: each is a module over the framework's linear layers (so d
 projections) that runs on rows of normed hidden states, a PagedKVCache and an AttnMeta.
 
 A mixer reads its sizes and constants from a spec and keeps what it remembers under its own run
-number of the cache: a layer that is run several times per token has one run per pass.
+number of the cache: a layer that is run several times per token has one run per pass.  `kind` says
+which pools ("kv", with `window`, None for all earlier tokens, and `shares`, the layer whose run it
+reads instead of one of its own; or "state"), `cache_shape` their sizes per token or sequence.
 `weight_views()` maps the mixer's checkpoint names (without the layer's prefix) to where they go."""
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Dict, List
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -94,10 +96,12 @@ def distance_bias(rel: torch.Tensor, bias_max: int, window: int) -> torch.Tensor
 
 class WindowAttention(nn.Module):
     kind = "kv"
+    shares = None
 
     def __init__(self, spec: WindowAttentionSpec, width: int, bias_rows: int, eps: float, device, dtype):
         super().__init__()
-        self.spec, self.eps = spec, eps
+        self.spec, self.eps, self.window = spec, eps, spec.window
+        self.cache_shape = (spec.kv_heads, spec.dim, spec.vdim)
         self.q_width, self.k_width = spec.heads * spec.dim, spec.kv_heads * spec.dim
         self.v_width = spec.kv_heads * spec.vdim
         self.qkv_proj = _stacked(width, self.q_width + self.k_width + self.v_width, device, dtype)
@@ -151,12 +155,14 @@ class MlstmSpec:
 
 class Mlstm(nn.Module):
     kind = "state"
+    normalised = True
     # portions up to this many tokens go through the recurrent kernel, longer ones 64 at a time
     RECURRENT_TOKENS = 4
 
     def __init__(self, spec: MlstmSpec, width: int, eps: float, device, dtype):
         super().__init__()
         self.spec, self.eps = spec, eps
+        self.cache_shape = (spec.heads, spec.dim, spec.vdim)
         self.qk, self.vw = spec.heads * spec.dim, spec.heads * spec.vdim
         self.qkvg_proj = _stacked(width, 2 * self.qk + 2 * self.vw, device, dtype)
         self.o_proj = L.RowParallelLinear(self.vw, width, device=device, dtype=dtype)
@@ -186,6 +192,242 @@ class Mlstm(nn.Module):
 
 
 # ---------------------------------------------------------------------------
+# attention over a cached latent
+# ---------------------------------------------------------------------------
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    heads: int
+    dim: int                            # query / key components per head without a rotation
+    rot_dim: int                        # ... and with one; a key's are shared by all heads
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+    kv_from: Optional[int] = None       # layer whose latents this one reads instead of its own
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "LatentAttentionSpec":
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d["rot_dim"]), int(d["vdim"]), int(d["kv_rank"]),
+                   float(d["scale"]), float(d["rot"]["base"]), None if d.get("kv_from") is None else int(d["kv_from"]))
+        if int(d["rot"]["dims"]) != spec.rot_dim or spec.rot_dim % 2:
+            raise ValueError("the rotation covers the rot_dim components, in pairs")
+        return spec
+
+
+@dataclass
+class _Rows:
+    """Some sequences of a batch and their rows."""
+    rows: Optional[torch.Tensor]        # row numbers, None: the slice [first, first + count)
+    first: int
+    count: int
+    max_query: int
+    q_starts: torch.Tensor
+    ctx_lens: torch.Tensor
+    block_tables: torch.Tensor
+    kv_starts: Optional[torch.Tensor] = None
+    total: int = 0                      # keys of all its sequences
+    longest: int = 0
+
+    def take(self, x: torch.Tensor) -> torch.Tensor:
+        return x[self.first:self.first + self.count] if self.rows is None else x[self.rows]
+
+    def put(self, out: torch.Tensor, part: torch.Tensor) -> None:
+        if self.rows is None:
+            out[self.first:self.first + self.count] = part
+        else:
+            out[self.rows] = part
+
+
+class LatentAttention(nn.Module):
+    """A token is cached as one row [latent | shared rotated key part].  Decoded tokens and short portions
+    take the queries to the latent (q W_uk, attention over the rows as they lie, then W_uv); longer portions
+    expand the rows of their sequences into keys and values of every head first."""
+    kind = "kv"
+    window = None
+    # portions up to this many tokens work on the latents directly
+    LATENT_TOKENS = 16
+    # most bytes of expanded keys and values at a time (a single sequence may exceed it)
+    EXPANDED_BYTES = 4 << 30
+
+    def __init__(self, spec: LatentAttentionSpec, width: int, eps: float, device, dtype):
+        super().__init__()
+        self.spec, self.eps, self.shares = spec, eps, spec.kv_from
+        self.row = spec.kv_rank + spec.rot_dim
+        self.cache_shape = (1, self.row, 0)
+        self.head = spec.dim + spec.rot_dim
+        self.q_width = spec.heads * self.head
+        own = self.shares is None
+        self.q_latent_proj = _stacked(width, self.q_width + (self.row if own else 0), device, dtype)
+        self.o_proj = L.RowParallelLinear(spec.heads * spec.vdim, width, device=device, dtype=dtype)
+        mat = lambda rows: nn.Parameter(torch.empty((rows, spec.kv_rank), dtype=dtype, device=device).normal_(
+            0, spec.kv_rank ** -0.5), requires_grad=False)
+        self.uk, self.uv = mat(spec.heads * spec.dim), mat(spec.heads * spec.vdim)
+        self.latent_norm = _vector(spec.kv_rank, device, 1.0) if own else None
+        self.sink = _vector(spec.heads, device)
+        self.expand = None
+
+    def weight_views(self) -> Dict[str, torch.Tensor]:
+        views = {"q": self.q_latent_proj.weight[: self.q_width], "uk": self.uk, "uv": self.uv, "sink": self.sink,
+                 "o": self.o_proj.weight}
+        if self.shares is None:
+            views["dkv"] = self.q_latent_proj.weight[self.q_width:self.q_width + self.row]
+            views["dkv.norm"] = self.latent_norm
+        return views
+
+    def prepare(self) -> None:
+        """The expansion of a cached row to [keys of all heads | values of all heads] as one matrix: a head's
+        key ends with the row's own shared part, which an identity block hands through unchanged."""
+        s = self.spec
+        w = torch.zeros((self.q_width + s.heads * s.vdim, self.row), dtype=self.uk.dtype, device=self.uk.device)
+        keys = w[: self.q_width].view(s.heads, self.head, self.row)
+        keys[:, : s.dim, : s.kv_rank] = self.uk.view(s.heads, s.dim, s.kv_rank)
+        keys[:, s.dim:, s.kv_rank:] = torch.eye(s.rot_dim, dtype=w.dtype, device=w.device)
+        w[self.q_width:, : s.kv_rank] = self.uv
+        self.expand = w
+        # 64-bit, so that a far position's angle is as good as a near one's
+        i = torch.arange(s.rot_dim // 2, dtype=torch.float64)
+        self.freq = (s.rot_base ** (-2.0 * i / s.rot_dim)).to(self.uk.device)
+
+    # -- which rows go which way -----------------------------------------------------------
+    def _split(self, meta: AttnMeta):
+        """(rows for the latent form or None, [groups of rows for the expanded form])."""
+        per_row = self.expand.shape[0] * self.expand.element_size()
+        most = max(1, self.EXPANDED_BYTES // per_row)
+        key = ("latent_attention", most, self.LATENT_TOKENS)
+        if key not in meta.shared:
+            meta.shared[key] = self._plan(meta, most)
+        return meta.shared[key]
+
+    def _plan(self, meta: AttnMeta, most: int):
+        dev = meta.q_starts.device
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        if meta.decode:
+            n = meta.ctx_lens.shape[0]
+            return _Rows(None, 0, n, 1, meta.q_starts, meta.ctx_lens, meta.block_tables), []
+        counts, ctx = meta.prompt_lens, meta.host_ctx_lens
+        starts = [0]
+        for n in counts:
+            starts.append(starts[-1] + n)
+
+        def pick(seqs: List[int]) -> _Rows:
+            lens, keys = [counts[i] for i in seqs], [ctx[i] + counts[i] for i in seqs]
+            first, total = starts[seqs[0]], sum(lens)
+            together = seqs == list(range(seqs[0], seqs[0] + len(seqs)))
+            rows = None if together else torch.tensor([r for i in seqs for r in range(starts[i], starts[i + 1])], device=dev)
+            edges = lambda v: i32([0] + torch.tensor(v).cumsum(0).tolist())
+            whole = len(seqs) == len(counts)
+            return _Rows(rows, first, total, max(lens), edges(lens), meta.ctx_lens if whole else i32([ctx[i] for i in seqs]),
+                         meta.block_tables if whole else meta.block_tables[torch.tensor(seqs, device=dev)], edges(keys),
+                         sum(keys), max(keys))
+
+        short = [i for i, n in enumerate(counts) if 0 < n <= self.LATENT_TOKENS]
+        groups: List[List[int]] = []
+        held = 0
+        for i, n in enumerate(counts):
+            if n > self.LATENT_TOKENS:
+                if not groups or held + ctx[i] + n > most:
+                    groups.append([])
+                    held = 0
+                groups[-1].append(i)
+                held += ctx[i] + n
+        return (pick(short) if short else None), [pick(g) for g in groups]
+
+    # -- forward ---------------------------------------------------------------------------
+    def _latent_form(self, part: _Rows, x: torch.Tensor, q: torch.Tensor, rows: torch.Tensor, block_size: int,
+                     out: torch.Tensor) -> None:
+        """x: rows with the queries; q [rows, heads, row]: their rotated components are in place."""
+        s = self.spec
+        plain = x[:, : self.q_width].unflatten(1, (s.heads, self.head))[..., : s.dim]
+        torch.bmm(plain.transpose(0, 1), self.uk.view(s.heads, s.dim, s.kv_rank), out=q[..., : s.kv_rank].transpose(0, 1))
+        o = ops.latent_attention(q, rows, part.block_tables, part.q_starts, part.ctx_lens, s.kv_rank, block_size, s.scale,
+                                 self.sink)
+        torch.bmm(o.transpose(0, 1), self.uv.view(s.heads, s.vdim, s.kv_rank).transpose(1, 2),
+                  out=out.view(-1, s.heads, s.vdim).transpose(0, 1))
+
+    def forward(self, h: torch.Tensor, cache: PagedKVCache, run: int, meta: AttnMeta) -> torch.Tensor:
+        s, rows, m = self.spec, cache.k[run], h.shape[0]
+        x = self.q_latent_proj(h)[0]
+        latent, groups = self._split(meta)
+        own = dict(l_off=self.q_width, norm_weight=self.latent_norm, eps=self.eps, cache=rows,
+                   slot_mapping=meta.slot_mapping) if self.shares is None else {}
+        q = x.new_empty((m, s.heads, self.row)) if not groups else None
+        ops.latent_rows(x, meta.positions, self.freq, s.heads, s.dim, s.rot_dim, s.kv_rank, q_out=q, **own)
+        att = x.new_empty((m, s.heads * s.vdim))
+        if latent is not None:
+            if q is not None:
+                self._latent_form(latent, x, q, rows, cache.block_size, att)
+            else:
+                part = latent.take(x)
+                q, o = x.new_empty((part.shape[0], s.heads, self.row)), x.new_empty((part.shape[0], att.shape[1]))
+                q[..., s.kv_rank:] = part[:, : self.q_width].unflatten(1, (s.heads, self.head))[..., s.dim:]
+                self._latent_form(latent, part, q, rows, cache.block_size, o)
+                latent.put(att, o)
+        for g in groups:
+            kv = ops.latent_gather(rows, g.block_tables, cache.block_size, g.kv_starts, g.total, g.longest)
+            kv = ops.base_gemm(kv, self.expand)
+            o = ops.rows_attention(g.take(x), kv, g.q_starts, g.ctx_lens, g.kv_starts, g.max_query, s.heads, s.heads,
+                                   self.head, s.vdim, s.scale, self.sink)
+            if g.count == m:
+                att = o
+            else:
+                g.put(att, o)
+        return self.o_proj(att)[0]
+
+
+# ---------------------------------------------------------------------------
+# linear attention with a constant decay
+# ---------------------------------------------------------------------------
+
+@dataclass(frozen=True)
+class LightningSpec:
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "LightningSpec":
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d["vdim"]), tuple(float(x) for x in d["decay"]))
+        if len(spec.decay) != spec.heads:
+            raise ValueError("one decay per head")
+        return spec
+
+
+class Lightning(nn.Module):
+    kind = "state"
+    normalised = False
+    # portions up to this many tokens go through the recurrent kernel, longer ones 64 at a time
+    RECURRENT_TOKENS = 4
+
+    def __init__(self, spec: LightningSpec, width: int, eps: float, device, dtype):
+        super().__init__()
+        self.spec, self.eps = spec, eps
+        self.cache_shape = (spec.heads, spec.dim, spec.vdim)
+        self.qk, self.vw = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.qkvg_proj = _stacked(width, 2 * self.qk + 2 * self.vw, device, dtype)
+        self.o_proj = L.RowParallelLinear(self.vw, width, device=device, dtype=dtype)
+        self.norm = _vector(self.vw, device, 1.0)
+        n = torch.arange(ops.LIGHTNING_POWERS, dtype=torch.float64)
+        self.powers = (torch.tensor(spec.decay, dtype=torch.float64)[:, None] ** n).float().to(device)
+        self.chunkwise = ops.lightning_chunk_supported(spec.dim, spec.vdim, dtype)
+
+    def weight_views(self) -> Dict[str, torch.Tensor]:
+        q, k, v, g = self.qkvg_proj.weight[: 2 * self.qk + 2 * self.vw].split([self.qk, self.qk, self.vw, self.vw])
+        return {"q": q, "k": k, "v": v, "g": g, "o": self.o_proj.weight, "norm": self.norm}
+
+    def prepare(self) -> None:
+        pass
+
+    def forward(self, h: torch.Tensor, cache: PagedKVCache, run: int, meta: AttnMeta) -> torch.Tensor:
+        st = cache.state
+        x = self.qkvg_proj(h)[0]
+        o = ops.lightning(x, self.powers, self.norm, st.S[run], meta.state_slots, meta.q_starts, meta.ctx_lens, self.eps,
+                          chunkwise=self.chunkwise and meta.max_query > self.RECURRENT_TOKENS)
+        return self.o_proj(o)[0]
+
+
+# ---------------------------------------------------------------------------
 # feed-forward
 # ---------------------------------------------------------------------------
 
@@ -204,3 +446,55 @@ class GatedMLP(nn.Module):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         return self.down_proj(ops.gated_act(self.gate_up_proj(h)[0], self.activation))[0]
+
+
+@dataclass(frozen=True)
+class RoutedExpertsSpec:
+    experts: int
+    top: int
+    ff: int
+    shared_ff: Optional[int] = None     # width of an expert that every token passes, None: there is none
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "RoutedExpertsSpec":
+        r, shared = d["router"], d.get("shared")
+        spec = cls(int(r["experts"]), int(r["top"]), int(d["expert"]["ff"]), int(shared["ff"]) if shared else None)
+        if not 1 <= spec.top <= spec.experts:
+            raise ValueError("a token takes between one and all of the experts")
+        return spec
+
+
+class RoutedExperts(nn.Module):
+    """Each token through its `top` experts down(act(up(s h))), s = sigmoid of the router's logit -- the score
+    scales the expert's input, which the up product's epilogue does to its result -- and, where there is
+    one, through a shared expert with scale 1.  Returns the shared expert's output and the routed rows,
+    which the next residual step sums."""
+
+    def __init__(self, spec: RoutedExpertsSpec, width: int, activation: str, device, dtype):
+        super().__init__()
+        self.spec, self.activation = spec, activation
+        mat = lambda *shape: nn.Parameter(torch.empty(shape, dtype=dtype, device=device).normal_(0, 0.02),
+                                          requires_grad=False)
+        self.router = mat(spec.experts, width)
+        self.up, self.down = mat(spec.experts, spec.ff, width), mat(spec.experts, width, spec.ff)
+        self.up_proj = self.down_proj = None
+        if spec.shared_ff is not None:
+            self.up_proj = _stacked(width, spec.shared_ff, device, dtype)
+            self.down_proj = L.RowParallelLinear(spec.shared_ff, width, device=device, dtype=dtype)
+
+    def weight_views(self) -> Dict[str, torch.Tensor]:
+        views = {"router": self.router}
+        for e in range(self.spec.experts):
+            views[f"e{e}.up"], views[f"e{e}.down"] = self.up[e], self.down[e]
+        if self.up_proj is not None:
+            views["shared.up"], views["shared.down"] = self.up_proj.weight[: self.spec.shared_ff], self.down_proj.weight
+        return views
+
+    def forward(self, h: torch.Tensor) -> ops.Update:
+        routing = ops.moe_route(ops.matmul_f32(h, self.router), self.spec.top)
+        a = ops.moe_gemm(ops.moe_gather(h, routing), self.up, routing.offsets, routing.sorted_scores, self.activation)
+        y = ops.moe_gemm(a, self.down, routing.offsets)
+        shared = None
+        if self.up_proj is not None:
+            shared = self.down_proj(ops.act(self.up_proj(h)[0], self.activation, self.spec.shared_ff))[0]
+        return ops.Update(shared, y, routing.place)

@@ -18,7 +18,7 @@ one for thousands of prompt tokens.
 from __future__ import annotations
 
 import ctypes
-from typing import Optional, Tuple
+from typing import NamedTuple, Optional, Tuple
 
 import torch
 
@@ -175,13 +175,14 @@ def _workspace(device, nbytes: int) -> torch.Tensor:
 
 
 def read_status(device=None) -> int:
-    """Reads and clears the status words the SBMM and the window attention kernels leave in the
+    """Reads and clears the status words the SBMM, window attention and expert kernels leave in the
     current stream's workspaces (0 = ok, DZ_ERR_TIMEOUT = a bounded device-side wait ran
     out, DZ_ERR_INVALID_ARG = a wrong `tokens_sorted` promise).  Synchronises."""
     device = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
     found = 0
     for ws in (_workspaces.get((device.index, _stream())),
-               _scratch.get(("window_attention", device.index, _stream()))):
+               _scratch.get(("window_attention", device.index, _stream())),
+               _scratch.get(("moe", device.index, _stream()))):
         if ws is not None:
             host = ctypes.c_int(0)
             check(lib().dz_read_status(ws.data_ptr(), _stream(), ctypes.byref(host)), "dz_read_status")
@@ -613,7 +614,7 @@ def paged_attention_decode(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: to
 # blocks, matrix-memory recurrence.  16-bit or 32-bit activations, any sizes.
 # ---------------------------------------------------------------------------
 
-ACTIVATIONS = {"silu": _lib.DZ_ACT_SILU, "gelu_tanh": _lib.DZ_ACT_GELU_TANH}
+ACTIVATIONS = {"silu": _lib.DZ_ACT_SILU, "gelu_tanh": _lib.DZ_ACT_GELU_TANH, "relu2": _lib.DZ_ACT_RELU2}
 _scratch = {}
 
 
@@ -646,27 +647,41 @@ def matmul_f32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     return torch.mm(x, weight.t(), out_dtype=torch.float32)
 
 
-def embed_norm(tokens: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float, weight_offset: float = 0.0,
-               copy: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """norm(table[tokens]) as a 32-bit residual [M, width]; `copy`: a column slice of a wider matrix
-    that gets the same rounded to the table's type."""
+def embed_norm(tokens: torch.Tensor, table: torch.Tensor, weight: Optional[torch.Tensor], eps: float,
+               weight_offset: float = 0.0, copy: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
+    """norm(scale * table[tokens]) as a 32-bit residual [M, width], without the norm when `weight` is None;
+    `copy`: a column slice of a wider matrix that gets the same rounded to the table's type."""
     _need_cuda(tokens, table, weight, copy)
     m, (vocab, width) = tokens.numel(), table.shape
     residual = torch.empty((m, width), dtype=torch.float32, device=table.device)
     if copy is not None and (copy.dtype != table.dtype or copy.shape != (m, width) or copy.stride(1) != 1):
         raise ValueError("copy must be a [tokens, width] slice of the table's type with unit column stride")
-    check(lib().dz_embed_norm(tokens.data_ptr(), table.data_ptr(), vocab, weight.data_ptr(), float(weight_offset),
+    check(lib().dz_embed_norm(tokens.data_ptr(), table.data_ptr(), vocab, float(scale), _ptr(weight), float(weight_offset),
                               residual.data_ptr(), _ptr(copy), copy.stride(0) if copy is not None else 0, m, width,
                               float(eps), _any_dtype_code(table), _stream()), "dz_embed_norm")
     return residual
 
 
-def residual_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float,
+class Update(NamedTuple):
+    """What a sublayer adds to the residual: a matrix, and optionally rows `index` [M, n] (int32, negative:
+    none) of a second one that are summed into each of its rows."""
+    matrix: Optional[torch.Tensor]
+    rows: Optional[torch.Tensor] = None
+    index: Optional[torch.Tensor] = None
+
+    def dense(self) -> torch.Tensor:
+        """The whole update in 32 bits (for inspection; residual_norm sums it on its way)."""
+        picked = torch.where(self.index[..., None] >= 0, self.rows[self.index.clamp(min=0).long()].float(), 0).sum(1)
+        return picked if self.matrix is None else picked + self.matrix
+
+
+def residual_norm(residual: torch.Tensor, delta, weight: Optional[torch.Tensor], eps: float,
                   dtype: torch.dtype, weight_offset: float = 0.0, vec: Optional[torch.Tensor] = None,
                   replace: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """residual (32-bit, in place) += delta + vec, or = with `replace`; returns norm(residual) in
-    `dtype`, or the residual rounded to it when `weight` is None."""
-    _need_cuda(residual, delta, weight, vec, out)
+    `dtype`, or the residual rounded to it when `weight` is None.  `delta`: a matrix, an Update or None."""
+    delta, rows, index = delta if isinstance(delta, Update) else (delta, None, None)
+    _need_cuda(residual, delta, weight, vec, out, rows, index)
     m, width = residual.shape
     if out is None:
         out = torch.empty((m, width), dtype=dtype, device=residual.device)
@@ -674,10 +689,24 @@ def residual_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight:
         raise ValueError("the residual is a contiguous float32 matrix, out has unit column stride")
     if delta is not None and (delta.shape != residual.shape or not delta.is_contiguous()):
         raise ValueError("delta must be a contiguous matrix of the residual's shape")
+    if rows is not None and (rows.dtype != out.dtype or rows.shape[1] != width or not rows.is_contiguous() or
+                             index.dtype != torch.int32 or index.shape[0] != m or not index.is_contiguous()):
+        raise ValueError("summed rows are contiguous, of the output's type, with an int32 index per row")
     check(lib().dz_residual_norm(residual.data_ptr(), _ptr(delta), _any_dtype_code(delta) if delta is not None else 0,
-                                 int(replace), _ptr(vec), _ptr(weight), float(weight_offset), out.data_ptr(),
+                                 int(replace), _ptr(vec), _ptr(rows), _ptr(index), index.shape[1] if rows is not None else 0,
+                                 _ptr(weight), float(weight_offset), out.data_ptr(),
                                  out.stride(0) if m > 1 else max(out.stride(0), width), m, width, float(eps),
                                  _any_dtype_code(out), _stream()), "dz_residual_norm")
+    return out
+
+
+def act(x: torch.Tensor, activation: str, inter: Optional[int] = None) -> torch.Tensor:
+    """act(x[:, :inter]); columns beyond are padding."""
+    _need_cuda(x)
+    inter = inter or x.shape[1]
+    out = torch.empty((x.shape[0], inter), dtype=x.dtype, device=x.device)
+    check(lib().dz_act(x.data_ptr(), x.stride(0), out.data_ptr(), x.shape[0], inter, ACTIVATIONS[activation],
+                       _any_dtype_code(x), _stream()), "dz_act")
     return out
 
 
@@ -715,10 +744,11 @@ def kv_append(qkv: torch.Tensor, k_off: int, k_cache: torch.Tensor, v_cache: tor
 def window_attention(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor,
                      q_starts: torch.Tensor, ctx_lens: torch.Tensor, max_query: int, decode: bool, heads: int,
                      block_size: int, scale: float, window: int, bias: Optional[torch.Tensor] = None,
-                     splits: int = 0) -> torch.Tensor:
+                     splits: int = 0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of [q | k | v | ...] rows with a sliding window and an additive bias per distance
-    ([heads, distances] float32); see dz_window_attention.  `splits` 0: enough CTAs to fill the GPU."""
-    _need_cuda(qkv, k_cache, v_cache, block_tables, q_starts, ctx_lens, bias)
+    ([heads, distances] float32); see dz_window_attention.  `splits` 0: enough CTAs to fill the GPU.
+    `sink` [heads] float32: one more score per row, without a key or a value."""
+    _need_cuda(qkv, k_cache, v_cache, block_tables, q_starts, ctx_lens, bias, sink)
     kv_heads, dim, vdim = k_cache.shape[1], k_cache.shape[2], v_cache.shape[2]
     rows, seqs = qkv.shape[0], ctx_lens.shape[0]
     if any(t.dtype != torch.int32 or not t.is_contiguous() for t in (block_tables, q_starts, ctx_lens)):
@@ -740,8 +770,136 @@ def window_attention(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Te
         q_starts=q_starts.data_ptr(), ctx_lens=ctx_lens.data_ptr(), num_seqs=seqs, rows=rows, max_q=max_query,
         decode=int(decode), heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=float(scale), window=window,
         bias=_ptr(bias), bias_len=bias.shape[1] if bias is not None else 0, splits=splits,
-        workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=_any_dtype_code(qkv))
+        workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=_any_dtype_code(qkv),
+        sink=_ptr(sink))
     check(lib().dz_window_attention(ctypes.byref(args), _stream()), "dz_window_attention")
+    return out
+
+
+def rows_attention(q: torch.Tensor, kv: torch.Tensor, q_starts: torch.Tensor, ctx_lens: torch.Tensor,
+                   kv_starts: torch.Tensor, max_query: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
+                   sink: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
+    """The same attention with every key and value of a sequence in rows [k | v | ...] of their own, its
+    position t in row kv_starts[sequence] + t (dz_window_attention with `kv`)."""
+    _need_cuda(q, kv, q_starts, ctx_lens, kv_starts, sink)
+    if any(t.dtype != torch.int32 or not t.is_contiguous() for t in (q_starts, ctx_lens, kv_starts)):
+        raise ValueError("q_starts / ctx_lens / kv_starts must be contiguous int32")
+    rows, seqs = q.shape[0], ctx_lens.shape[0]
+    out = torch.empty((rows, heads * vdim), dtype=q.dtype, device=q.device)
+    ws = _zeroed_scratch("window_attention", q.device, lib().dz_window_attention_workspace_bytes(seqs, heads, kv_heads, vdim, 1))
+    args = _lib.WindowAttentionArgs(
+        qkv=q.data_ptr(), row_stride=q.stride(0), k_off=0, v_off=kv_heads * dim, out=out.data_ptr(),
+        q_starts=q_starts.data_ptr(), ctx_lens=ctx_lens.data_ptr(), num_seqs=seqs, rows=rows, max_q=max_query, decode=0,
+        heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=float(scale), window=window, splits=1,
+        workspace=ws.data_ptr(), workspace_bytes=ws.numel(), dtype=_any_dtype_code(q), sink=_ptr(sink), kv=kv.data_ptr(),
+        kv_stride=kv.stride(0), kv_starts=kv_starts.data_ptr(), kv_rows=kv.shape[0])
+    check(lib().dz_window_attention(ctypes.byref(args), _stream()), "dz_window_attention")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# attention over a cached latent, one row [latent | shared rotated key part] per token
+# ---------------------------------------------------------------------------
+
+def latent_rows(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, heads: int, dim: int, rot: int, rank: int,
+                q_out: Optional[torch.Tensor] = None, l_off: int = -1, norm_weight: Optional[torch.Tensor] = None,
+                eps: float = 0.0, cache: Optional[torch.Tensor] = None, slot_mapping: Optional[torch.Tensor] = None) -> None:
+    """Rotates the queries' last `rot` components (in place, or into the end of q_out's rows) and, with
+    l_off >= 0, writes the rows' normed latent and rotated key part to the cache (dz_latent_rows)."""
+    _need_cuda(x, positions, freq, q_out, norm_weight, cache, slot_mapping)
+    if positions.dtype != torch.int64 or freq.dtype != torch.float64 or freq.numel() != rot // 2:
+        raise ValueError("positions are int64, freq holds rot / 2 float64 values")
+    if q_out is not None and (q_out.shape != (x.shape[0], heads, rank + rot) or not q_out.is_contiguous()):
+        raise ValueError("q_out must be a contiguous [rows, heads, rank + rot]")
+    args = _lib.LatentRowsArgs(
+        x=x.data_ptr(), row_stride=x.stride(0), positions=positions.data_ptr(), freq=freq.data_ptr(), rows=x.shape[0],
+        heads=heads, dim=dim, rot=rot, q_out=_ptr(q_out), l_off=l_off, rank=rank, norm_weight=_ptr(norm_weight),
+        eps=float(eps), cache=_ptr(cache), slots=_ptr(slot_mapping), dtype=_any_dtype_code(x))
+    check(lib().dz_latent_rows(ctypes.byref(args), _stream()), "dz_latent_rows")
+
+
+def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, block_size: int, starts: torch.Tensor, total: int,
+                  max_len: int) -> torch.Tensor:
+    """Cached rows of positions 0, 1, ... of every sequence, sequence after sequence: [total, row size]."""
+    _need_cuda(cache, block_tables, starts)
+    size = cache.shape[-1]
+    out = torch.empty((total, size), dtype=cache.dtype, device=cache.device)
+    check(lib().dz_latent_gather(cache.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], block_size,
+                                 starts.data_ptr(), block_tables.shape[0], max_len, out.data_ptr(), size,
+                                 _any_dtype_code(cache), _stream()), "dz_latent_gather")
+    return out
+
+
+def _balanced_splits(ctas: int, most: int, sms: int = 148) -> int:
+    """Splits of every CTA's work with the fullest last wave; fewer where that gains little."""
+    best, score = 1, 0.0
+    for s in range(1, max(1, most) + 1):
+        full = ctas * s / (-(-ctas * s // sms) * sms)
+        if full > score * 1.05:
+            best, score = s, full
+    return best
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, q_starts: torch.Tensor,
+                     ctx_lens: torch.Tensor, rank: int, block_size: int, scale: float, sink: Optional[torch.Tensor] = None,
+                     splits: int = 0) -> torch.Tensor:
+    """q [rows, heads, rank + rot] against the cached rows up to each row's position; returns the weighted
+    latents [rows, heads, rank] (dz_latent_attention).  `splits` 0: chosen to fill the GPU."""
+    _need_cuda(q, cache, block_tables, q_starts, ctx_lens, sink)
+    rows, heads, size = q.shape
+    if not q.is_contiguous() or cache.shape[-1] != size or not cache.is_contiguous():
+        raise ValueError("q is a contiguous [rows, heads, rank + rot] with the cache's row size")
+    if any(t.dtype != torch.int32 or not t.is_contiguous() for t in (block_tables, q_starts, ctx_lens)):
+        raise ValueError("block_tables / q_starts / ctx_lens must be contiguous int32")
+    code = _any_dtype_code(q)
+    ctas = lib().dz_latent_attention_ctas(rows, heads, rank, size - rank, code)
+    if ctas == 0:
+        splits = 1
+    elif splits <= 0:
+        splits = _balanced_splits(ctas, min(16, -(-block_tables.shape[1] * block_size // 256)))
+    out = torch.empty((rows, heads, rank), dtype=q.dtype, device=q.device)
+    ws = _zeroed_scratch("latent_attention", q.device, lib().dz_latent_attention_workspace_bytes(rows, heads, rank, splits))
+    args = _lib.LatentAttentionArgs(
+        q=q.data_ptr(), cache=cache.data_ptr(), block_tables=block_tables.data_ptr(), table_width=block_tables.shape[1],
+        block_size=block_size, q_starts=q_starts.data_ptr(), ctx_lens=ctx_lens.data_ptr(), num_seqs=ctx_lens.shape[0],
+        rows=rows, heads=heads, rank=rank, rot=size - rank, scale=float(scale), sink=_ptr(sink), out=out.data_ptr(),
+        splits=splits, workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=code)
+    check(lib().dz_latent_attention(ctypes.byref(args), _stream()), "dz_latent_attention")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# recurrent layers
+# ---------------------------------------------------------------------------
+
+LIGHTNING_POWERS = 65                   # decay^0 ... decay^64 per head
+
+
+def lightning_chunk_supported(dim: int, vdim: int, dtype: torch.dtype) -> bool:
+    code = {torch.float16: _lib.DZ_DTYPE_F16, torch.bfloat16: _lib.DZ_DTYPE_BF16}.get(dtype, _lib.DZ_DTYPE_F32)
+    return bool(lib().dz_lightning_chunk_supported(dim, vdim, code))
+
+
+def lightning(x: torch.Tensor, powers: torch.Tensor, norm_weight: torch.Tensor, S: torch.Tensor, slots: torch.Tensor,
+              q_starts: torch.Tensor, ctx_lens: torch.Tensor, eps: float, chunkwise: bool) -> torch.Tensor:
+    """Linear attention with a constant decay, norm over all heads and output gate over rows
+    [q | k | v | g | ...]; the states in slots `slots` are updated in place (dz_lightning)."""
+    _need_cuda(x, powers, norm_weight, S, slots, q_starts, ctx_lens)
+    heads, dim, vdim = S.shape[1:]
+    rows, seqs = x.shape[0], ctx_lens.shape[0]
+    if any(t.dtype != torch.int32 or not t.is_contiguous() for t in (slots, q_starts, ctx_lens)):
+        raise ValueError("slots / q_starts / ctx_lens must be contiguous int32")
+    if powers.shape != (heads, LIGHTNING_POWERS) or powers.dtype != torch.float32 or not powers.is_contiguous():
+        raise ValueError("powers must be a contiguous float32 [heads, 65]")
+    out = torch.empty((rows, heads * vdim), dtype=x.dtype, device=x.device)
+    ws = _zeroed_scratch("lightning", x.device, lib().dz_lightning_workspace_bytes(rows, seqs, heads, vdim, int(chunkwise)))
+    args = _lib.LightningArgs(
+        x=x.data_ptr(), row_stride=x.stride(0), k_off=heads * dim, v_off=2 * heads * dim,
+        g_off=2 * heads * dim + heads * vdim, powers=powers.data_ptr(), norm_weight=norm_weight.data_ptr(),
+        eps=float(eps), out=out.data_ptr(), S=S.data_ptr(), slots=slots.data_ptr(), q_starts=q_starts.data_ptr(),
+        ctx_lens=ctx_lens.data_ptr(), num_seqs=seqs, rows=rows, heads=heads, dim=dim, vdim=vdim, chunkwise=int(chunkwise),
+        workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=_any_dtype_code(x))
+    check(lib().dz_lightning(ctypes.byref(args), _stream()), "dz_lightning")
     return out
 
 
@@ -772,4 +930,61 @@ def mlstm(x: torch.Tensor, h: torch.Tensor, w_if: torch.Tensor, b_if: torch.Tens
         num_seqs=seqs, rows=rows, heads=heads, dim=dim, vdim=vdim, chunkwise=int(chunkwise),
         workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=_any_dtype_code(x))
     check(lib().dz_mlstm(ctypes.byref(args), _stream()), "dz_mlstm")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# routed experts
+# ---------------------------------------------------------------------------
+
+class Routing(NamedTuple):
+    """Entries (token, choice) of a batch in expert order."""
+    ids: torch.Tensor                   # int32 [M, top] chosen experts
+    scores: torch.Tensor                # float32 [M, top]
+    offsets: torch.Tensor               # int32 [experts + 1] first sorted row of every expert
+    place: torch.Tensor                 # int32 [M, top] sorted row of an entry
+    order: torch.Tensor                 # int32 [M * top] entry of a sorted row
+    sorted_scores: torch.Tensor         # float32 [M * top]
+
+
+def moe_route(logits: torch.Tensor, top: int) -> Routing:
+    """The `top` experts of every token by sigmoid(logits), and the batch's entries sorted by expert."""
+    _need_cuda(logits)
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise ValueError("router logits are contiguous float32")
+    m, experts = logits.shape
+    dev, i32 = logits.device, torch.int32
+    ids, place = (torch.empty((m, top), dtype=i32, device=dev) for _ in range(2))
+    scores = torch.empty((m, top), dtype=torch.float32, device=dev)
+    offsets, order = torch.empty(experts + 1, dtype=i32, device=dev), torch.empty(m * top, dtype=i32, device=dev)
+    by_expert = torch.empty(m * top, dtype=torch.float32, device=dev)
+    check(lib().dz_moe_route(logits.data_ptr(), m, experts, top, ids.data_ptr(), scores.data_ptr(), _stream()), "dz_moe_route")
+    check(lib().dz_moe_sort(ids.data_ptr(), scores.data_ptr(), m * top, experts, offsets.data_ptr(), place.data_ptr(),
+                            order.data_ptr(), by_expert.data_ptr(), _stream()), "dz_moe_sort")
+    return Routing(ids, scores, offsets, place, order, by_expert)
+
+
+def moe_gather(x: torch.Tensor, routing: Routing) -> torch.Tensor:
+    """The entries' token rows in expert order."""
+    _need_cuda(x)
+    entries, top = routing.order.numel(), routing.ids.shape[1]
+    out = torch.empty((entries, x.shape[1]), dtype=x.dtype, device=x.device)
+    check(lib().dz_moe_gather(x.data_ptr(), routing.order.data_ptr(), entries, top, out.data_ptr(), x.shape[1],
+                              _any_dtype_code(x), _stream()), "dz_moe_gather")
+    return out
+
+
+def moe_gemm(x: torch.Tensor, weights: torch.Tensor, offsets: torch.Tensor, scale: Optional[torch.Tensor] = None,
+             activation: Optional[str] = None) -> torch.Tensor:
+    """act(scale * (x W_e^T)) for rows x in expert order, weights [experts, N, K]."""
+    _need_cuda(x, weights, offsets, scale)
+    experts, n, k = weights.shape
+    rows = x.shape[0]
+    if x.shape[1] != k or not x.is_contiguous() or not weights.is_contiguous() or x.dtype != weights.dtype:
+        raise ValueError("x [rows, K] and weights [experts, N, K] must be contiguous and of one type")
+    out = torch.empty((rows, n), dtype=x.dtype, device=x.device)
+    status = _zeroed_scratch("moe", x.device, 256)
+    check(lib().dz_moe_gemm(x.data_ptr(), weights.data_ptr(), offsets.data_ptr(), _ptr(scale), out.data_ptr(), rows, n, k,
+                            experts, ACTIVATIONS[activation] if activation else _lib.DZ_ACT_NONE, -(-rows // experts),
+                            _any_dtype_code(x), status.data_ptr(), _stream()), "dz_moe_gemm")
     return out

@@ -10,6 +10,7 @@ import torch
 from . import loader
 from .buzalorn import BuzalornConfig, BuzalornForCausalLM
 from .llama import LlamaConfig, LlamaForCausalLM
+from .movarax import MovaraxConfig, MovaraxForCausalLM
 
 
 @dataclass(frozen=True)
@@ -40,6 +41,8 @@ register(ModelEntry("LlamaForCausalLM", LlamaConfig, LlamaForCausalLM, torch.flo
                     (torch.float16, torch.bfloat16), _llama_from_tensors))
 register(ModelEntry("Buzalorn", BuzalornConfig, BuzalornForCausalLM, torch.bfloat16,
                     (torch.float16, torch.bfloat16, torch.float32), BuzalornForCausalLM.from_tensors))
+register(ModelEntry("Movarax", MovaraxConfig, MovaraxForCausalLM, torch.bfloat16,
+                    (torch.float16, torch.bfloat16, torch.float32), MovaraxForCausalLM.from_tensors))
 
 
 def names():

@@ -309,21 +309,28 @@ int dz_pack_gptq(const float* Wq, const float* scale, const float* zero, int N, 
  * A norm is x / sqrt(mean(x^2) + eps) * (weight_offset + weight), weights in 32 bits: offset 0 is the
  * plain RMS norm, 1 the form whose weight is stored around zero.
  *
- *   embed_norm     residual = norm(table[token]); with `copy`, the same rounded to dtype goes to a
- *                  column slice of a wider matrix (copy_stride elements per row)
+ *   embed_norm     residual = norm(scale * table[token]), without the norm where weight is NULL; with
+ *                  `copy`, the same rounded to dtype goes to a column slice of a wider matrix
+ *                  (copy_stride elements per row)
  *   residual_norm  residual = (replace ? 0 : residual) + delta + vec; out = norm(residual), or the
  *                  residual itself when weight is NULL.  delta: dtype or DZ_DTYPE_F32; delta and vec
- *                  may be NULL
+ *                  may be NULL.  sum_count > 0: rows sum_index[r * sum_count + j] of sum_rows [*, width]
+ *                  (dtype) are added to row r as well (index < 0: none)
  *   gated_act      out[m, i] = act(x[m, i]) * x[m, inter + i]
+ *   act            out[m, i] = act(x[m, i])
+ * Activations: SiLU, GELU with tanh, max(z, 0)^2.
  */
 #define DZ_ACT_SILU 0
 #define DZ_ACT_GELU_TANH 1
-int dz_embed_norm(const int64_t* tokens, const void* table, int64_t vocab, const float* weight, float weight_offset,
-                  float* residual, void* copy, int64_t copy_stride, int M, int width, float eps, int dtype,
-                  void* stream);
+#define DZ_ACT_RELU2 2
+int dz_embed_norm(const int64_t* tokens, const void* table, int64_t vocab, float scale, const float* weight,
+                  float weight_offset, float* residual, void* copy, int64_t copy_stride, int M, int width, float eps,
+                  int dtype, void* stream);
 int dz_residual_norm(float* residual, const void* delta, int delta_dtype, int replace, const float* vec,
-                     const float* weight, float weight_offset, void* out, int64_t out_stride, int M, int width,
-                     float eps, int dtype, void* stream);
+                     const void* sum_rows, const int32_t* sum_index, int sum_count, const float* weight,
+                     float weight_offset, void* out, int64_t out_stride, int M, int width, float eps, int dtype,
+                     void* stream);
+int dz_act(const void* x, int64_t x_stride, void* out, int M, int inter, int act, int dtype, void* stream);
 int dz_gated_act(const void* x, int64_t x_stride, void* out, int M, int inter, int act, int dtype, void* stream);
 
 /*
@@ -336,6 +343,10 @@ int dz_gated_act(const void* x, int64_t x_stride, void* out, int M, int inter, i
  * are appended with dz_kv_append afterwards; decode = 1 (one row per sequence): the row's key and
  * value are in the cache already (dz_qk_norm with slot_mapping).  With splits > 1 the workspace must
  * be zero-filled once before its first use.
+ *
+ * With `kv` (decode = 0 only) every key and value of a sequence, from position 0 on, lies in kv_rows
+ * rows of its own, position t in row kv_starts[s] + t, columns k_off and v_off; the cache is not read.
+ * `sink` (float [heads], may be NULL): the softmax's denominator has one more term exp(sink[head]).
  */
 typedef struct dz_window_attention_args {
   const void* qkv;
@@ -357,6 +368,11 @@ typedef struct dz_window_attention_args {
   void* workspace;
   size_t workspace_bytes;
   int32_t dtype;
+  const float* sink;
+  const void* kv;
+  int64_t kv_stride;
+  const int32_t* kv_starts;
+  int32_t kv_rows;
 } dz_window_attention_args;
 size_t dz_window_attention_workspace_bytes(int num_seqs, int heads, int kv_heads, int vdim, int splits);
 int dz_window_attention(const dz_window_attention_args* args, void* stream);
@@ -403,6 +419,108 @@ typedef struct dz_mlstm_args {
 int dz_mlstm_chunk_supported(int dim, int vdim, int dtype);
 size_t dz_mlstm_workspace_bytes(int num_seqs, int heads);
 int dz_mlstm(const dz_mlstm_args* args, void* stream);
+
+/*
+ * Attention over a cached latent (dz_latent.cu).  A token's cache row is [c (rank) | r (rot)].
+ *
+ *   latent_rows       per row of x: the last rot of every head's dim + rot query components are rotated
+ *                     (in place, or into the last rot columns of q_out [rows, heads, rank + rot]); with
+ *                     l_off >= 0 the rank + rot columns from there are the token's own latent (RMS norm,
+ *                     plain weight) and shared key part (rotated), written to cache row slots[r] (< 0:
+ *                     not kept).  Neighbours (2i, 2i + 1) turn by positions[r] * freq[i], freq in 64 bits
+ *   latent_gather     cache rows of positions 0, 1, ... of sequence s to out rows starts[s] ... starts[s + 1]
+ *   latent_attention  q [rows, heads, rank + rot] against the cache rows of the row's sequence up to its
+ *                     own position (which must be there already): softmax(q.[c|r] * scale, with one more
+ *                     term exp(sink[head]) where sink is given) times c, [rows, heads, rank].  Row r of
+ *                     sequence s has position ctx_lens[s] + r - q_starts[s].  With splits > 1 the
+ *                     workspace must be zero-filled once before its first use
+ */
+typedef struct dz_latent_rows_args {
+  const void* x;
+  int64_t row_stride;
+  const int64_t* positions;
+  const double* freq;
+  int32_t rows, heads, dim, rot;
+  void* q_out;
+  int32_t l_off, rank;
+  const float* norm_weight;
+  float eps;
+  void* cache;
+  const int64_t* slots;
+  int32_t dtype;
+} dz_latent_rows_args;
+int dz_latent_rows(const dz_latent_rows_args* args, void* stream);
+int dz_latent_gather(const void* cache, const int32_t* block_tables, int table_width, int block_size, const int32_t* starts,
+                     int num_seqs, int max_len, void* out, int row_size, int dtype, void* stream);
+typedef struct dz_latent_attention_args {
+  const void* q;
+  const void* cache;
+  const int32_t* block_tables;
+  int32_t table_width, block_size;
+  const int32_t* q_starts;
+  const int32_t* ctx_lens;
+  int32_t num_seqs, rows, heads, rank, rot;
+  float scale;
+  const float* sink;
+  void* out;
+  int32_t splits;
+  void* workspace;
+  size_t workspace_bytes;
+  int32_t dtype;
+} dz_latent_attention_args;
+int dz_latent_attention_ctas(int rows, int heads, int rank, int rot, int dtype);
+size_t dz_latent_attention_workspace_bytes(int rows, int heads, int rank, int splits);
+int dz_latent_attention(const dz_latent_attention_args* args, void* stream);
+
+/*
+ * Linear attention with a constant decay per head (dz_lightning.cu): S <- decay S + k v^T, o = S^T q,
+ * with q, k, v = SiLU of the rows' [q | k | v] parts; then out = RMS norm over all heads' o together
+ * (plain weight) * sigmoid(g).  Rows are [q | k | v | g] (heads * dim, heads * dim, heads * vdim,
+ * heads * vdim); S [slots, heads, dim, vdim] is 32-bit and updated in place; a sequence with ctx_lens 0
+ * starts from zero without reading its slot.  powers [heads, 65]: decay^0 ... decay^64.
+ * chunkwise = 1 (dz_lightning_chunk_supported): 64 tokens at a time.  The workspace must be zero-filled
+ * once before its first use.
+ */
+typedef struct dz_lightning_args {
+  const void* x;
+  int64_t row_stride;
+  int32_t k_off, v_off, g_off;
+  const float* powers;
+  const float* norm_weight;
+  float eps;
+  void* out;
+  float* S;
+  const int32_t* slots;
+  const int32_t* q_starts;
+  const int32_t* ctx_lens;
+  int32_t num_seqs, rows, heads, dim, vdim, chunkwise;
+  void* workspace;
+  size_t workspace_bytes;
+  int32_t dtype;
+} dz_lightning_args;
+int dz_lightning_chunk_supported(int dim, int vdim, int dtype);
+size_t dz_lightning_workspace_bytes(int rows, int num_seqs, int heads, int vdim, int chunkwise);
+int dz_lightning(const dz_lightning_args* args, void* stream);
+
+/*
+ * Routed experts (dz_moe.cu).  An entry is one (token, choice), number token * top + choice; sorted
+ * entries lie expert by expert, in entry order within an expert.
+ *
+ *   moe_route   the top experts of every token by sigmoid(logits) (ties: the lower number) and their scores
+ *   moe_sort    offsets [experts + 1]: first sorted row of every expert; place [entries]: sorted row of an
+ *               entry (-1 for an id outside the range); order [entries]: entry of a sorted row (-1: none);
+ *               sorted_scores
+ *   moe_gather  out[row] = x[order[row] / top]
+ *   moe_gemm    y[row] = act(scale[row] * (x[row] W_e^T)) for the rows of expert e, weights [experts, N, K];
+ *               scale may be NULL, act DZ_ACT_NONE or an activation; `typical`: rows per expert to tile for
+ */
+#define DZ_ACT_NONE (-1)
+int dz_moe_route(const float* logits, int M, int experts, int top, int32_t* ids, float* scores, void* stream);
+int dz_moe_sort(const int32_t* ids, const float* scores, int entries, int experts, int32_t* offsets, int32_t* place,
+                int32_t* order, float* sorted_scores, void* stream);
+int dz_moe_gather(const void* x, const int32_t* order, int entries, int top, void* out, int width, int dtype, void* stream);
+int dz_moe_gemm(const void* x, const void* weights, const int32_t* offsets, const float* scale, void* y, int rows, int N,
+                int K, int experts, int act, int typical, int dtype, int* status, void* stream);
 
 /*
  * Delta swap-in: one asynchronous host->device copy of a delta's slot bytes
