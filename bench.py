@@ -17,8 +17,9 @@ request-to-delta map, tensor parallel.  --config 5: Llama-2-70B, 16 4-bit deltas
 memory, 4 GPU slots, bursty arrivals, swap-in overlapped with decode (--duration seconds of
 arrivals on a virtual clock).
 
---arch buzalorn: prefill and decode throughput of the Buzalorn decoder beside the Llama decoder at
-equal sizes, and the kernels of both against their rooflines (deltazip_b200/model_bench.py).
+--arch buzalorn | movarax: prefill and decode throughput of the Buzalorn decoder beside the Llama
+decoder, or of the Movarax decoder beside the Buzalorn one, at equal sizes, and the kernels of both
+against their rooflines (deltazip_b200/model_bench.py).
 
 N > 1: tensor parallel over N ranks (column-parallel qkv / gate_up, row-parallel o / down
 followed by the library's peer-memory all-reduce), shards cut at whole 128-wide units; the total
@@ -1282,9 +1283,9 @@ def main():
                     help="config 5: seconds of simulated arrivals (default 300)")
     ap.add_argument("--wall-limit", type=float, default=None,
                     help="config 5: stop the serving loop after this many wall-clock seconds (default 600)")
-    ap.add_argument("--arch", default=None, choices=["buzalorn"],
-                    help="instead of a configuration: this decoder beside the Llama decoder at equal sizes, whole "
-                         "models and kernel by kernel")
+    ap.add_argument("--arch", default=None, choices=["buzalorn", "movarax"],
+                    help="instead of a configuration: this decoder beside its closest one (Llama, Buzalorn) at equal "
+                         "sizes, whole models and kernel by kernel")
     ap.add_argument("--size", default=None, help="--arch: only these sizes (comma-separated)")
     args = ap.parse_args()
     if args.arch:

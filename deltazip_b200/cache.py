@@ -92,6 +92,12 @@ class PagedKVCache:
         if self.state is not None:
             seq.state_slot = self.state.allocate()
 
+    def reserve(self, seq, tokens: int) -> None:
+        """Gives an open `seq` the blocks it still lacks for `tokens` tokens.  (A ring has all it will ever
+        have: its positions are counted modulo its blocks.)"""
+        if self.window is None and len(seq.blocks) < self.blocks_for(tokens):
+            seq.blocks = seq.blocks + self.allocate(self.blocks_for(tokens) - len(seq.blocks))
+
     def close(self, seq) -> None:
         self.release(seq.blocks)
         seq.blocks = []

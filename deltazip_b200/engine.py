@@ -267,9 +267,12 @@ class DecodeEngine:
     @torch.inference_mode()
     def extend(self, work: List[Tuple[Sequence, List[int]]]) -> torch.Tensor:
         """Runs the given next tokens of admitted sequences (new prompts, portions of prompts, single
-        tokens, in any mixture) from the cache and state that earlier calls left.  Returns the hidden
-        states of all the tokens, in the order of `work`.  Models that support it take long
-        work in passes of at most `max_prefill_tokens` rows."""
+        tokens, in any mixture) from the cache and state that earlier calls left; a sequence that was
+        admitted for fewer tokens takes further cache blocks.  Returns the hidden states of all the
+        tokens, in the order of `work`.  Models that support it take long work in passes of at most
+        `max_prefill_tokens` rows."""
+        for s, toks in work:
+            self.cache.reserve(s, s.length + len(toks))
         order = sorted(range(len(work)), key=lambda i: self._sort_key(work[i][0]))
         limit = self.max_prefill_tokens if self.model.supports_portions else None
         parts: List[List[torch.Tensor]] = [[] for _ in work]

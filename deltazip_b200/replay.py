@@ -35,13 +35,15 @@ class Replayer:
         if want not in registry.lookup(loader.read_config(model_dir)).dtypes:
             raise NotImplementedError(f"this model does not run in {dtype}")
         cfg, model = registry.load_model(model_dir, device=device, dtype=want)
-        self.max_tokens = max(1, max_tokens)
         window = getattr(model, "window", None)
-        per_seq = -(-min(self.max_tokens, window if window is not None else self.max_tokens) // BLOCK)
-        # windowed models: room for every request's ring; others: for max_tokens in all
-        blocks = per_seq * MAX_SEQS if window is not None else per_seq
+        if window is not None:                  # room for every request's ring, which is opened at its full size
+            self.open_tokens = max(1, max_tokens)
+            blocks = -(-min(self.open_tokens, window) // BLOCK) * MAX_SEQS
+        else:                                   # room for max_tokens in all; requests take blocks as they grow
+            self.open_tokens = 0
+            blocks = -(-max(1, max_tokens) // BLOCK) + MAX_SEQS
         self.engine = DecodeEngine(cfg, None, MAX_SEQS, max(1, blocks), BLOCK, device=device, model=model)
-        self.live = {}
+        self.live, self.opened = {}, 0
 
     def step(self, entries: list):
         """Runs one step; returns the wanted logits on the host or None."""
@@ -50,7 +52,8 @@ class Replayer:
         for e in entries:
             seq = self.live.get(e["id"])
             if seq is None:
-                seq = self.live[e["id"]] = self.Sequence(len(self.live), 0, 0, self.max_tokens)
+                seq = self.live[e["id"]] = self.Sequence(self.opened, 0, 0, self.open_tokens)
+                self.opened += 1
                 if not eng.admit([seq]):
                     raise RuntimeError("the cache has no room for another request")
             work.append((seq, e["tokens"]))

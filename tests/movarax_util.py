@@ -90,7 +90,7 @@ def make_tensors(config, seed=0):
         n = mlp["router"]["experts"]
         t[p + "norm2"][:codes] = 1.0
         reads = torch.randperm(codes, generator=g)[:n]
-        router = torch.randn((n, w), generator=g) * 0.01
+        router = torch.randn((n, w), generator=g) * 0.003
         router[:, :codes] = 0
         router[torch.arange(n), reads] = 2.0
         t[p + "mlp.router"] = router.to(torch.bfloat16)
