@@ -487,9 +487,8 @@ int dz_rotary_and_cache(void* qkv, const int64_t* positions, const int64_t* slot
 
 size_t dz_paged_attention_workspace_bytes(int num_seqs, int q_heads, int kv_heads, int splits) {
   if (num_seqs <= 0 || q_heads <= 0 || kv_heads <= 0 || splits <= 0) return 0;
-  // tickets (rounded to 256 bytes) + partial triples
-  const size_t tickets = (((size_t)num_seqs * kv_heads * 4) + 255) & ~(size_t)255;
-  return tickets + (splits > 1 ? (size_t)num_seqs * q_heads * splits * (kHeadDim + 2) * 4 : 0);
+  // tickets + partial triples
+  return kTicketBytes + (splits > 1 ? (size_t)num_seqs * q_heads * splits * (kHeadDim + 2) * 4 : 0);
 }
 
 int dz_paged_attention_decode(const void* qkv, int q_row_stride, void* out, const void* k_cache,
@@ -513,8 +512,8 @@ int dz_paged_attention_decode(const void* qkv, int q_row_stride, void* out, cons
     if (!workspace || workspace_bytes < dz_paged_attention_workspace_bytes(num_seqs, q_heads, kv_heads, splits))
       return DZ_ERR_WORKSPACE;
     tickets = reinterpret_cast<int*>(workspace);
-    partial = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(workspace) +
-                                       ((((size_t)num_seqs * kv_heads * 4) + 255) & ~(size_t)255));
+    partial = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(workspace) + kTicketBytes);
+    if ((int64_t)num_seqs * kv_heads > kMaxTickets) return DZ_ERR_TOO_LARGE;
   }
   cudaStream_t st = (cudaStream_t)stream;
   const dim3 grid(kv_heads, num_seqs, splits);

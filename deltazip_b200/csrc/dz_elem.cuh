@@ -175,6 +175,12 @@ template <typename K> inline cudaError_t allow_smem(K kern, size_t bytes) {
 }
 constexpr size_t kMaxDynSmem = 220 * 1024;
 
+// Workspaces that hold both tickets (zero between launches) and other scratch start with the tickets,
+// and with room for this many whatever the launch needs: no launch's scratch may lie where the tickets of
+// another one of the same workspace are.
+constexpr int kMaxTickets = 65536;
+constexpr size_t kTicketBytes = (size_t)kMaxTickets * 4;
+
 inline bool is_float_dtype(int d) { return d == DZ_DTYPE_F16 || d == DZ_DTYPE_BF16 || d == DZ_DTYPE_F32; }
 
 }  // namespace dz

@@ -409,7 +409,6 @@ size_t latent_smem(int heads, int d) {
   const size_t h = 16 * head_tiles(heads), ld = (d + 15) / 16 * 16 + 8;
   return (h + 2 * kKeys) * ld * 2 + 2 * h * kLdP * 2 + 2 * h * kLdS * 4;
 }
-size_t latent_ticket_bytes(int rows, int heads) { return ((size_t)rows * head_groups(heads) * 4 + 255) & ~(size_t)255; }
 
 bool tensor_core_shapes(int heads, int rank, int rot, int dtype) {
   return (dtype == DZ_DTYPE_F16 || dtype == DZ_DTYPE_BF16) && rank % 8 == 0 && (rank + rot) % 8 == 0 &&
@@ -479,7 +478,7 @@ int dz_latent_attention_ctas(int rows, int heads, int rank, int rot, int dtype) 
 
 size_t dz_latent_attention_workspace_bytes(int rows, int heads, int rank, int splits) {
   if (rows <= 0 || heads <= 0 || rank <= 0 || splits <= 1) return 0;
-  return latent_ticket_bytes(rows, heads) + (size_t)rows * heads * splits * (rank + 2) * 4;
+  return kTicketBytes + (size_t)rows * heads * splits * (rank + 2) * 4;
 }
 
 int dz_latent_attention(const dz_latent_attention_args* a, void* stream) {
@@ -519,7 +518,8 @@ int dz_latent_attention(const dz_latent_attention_args* a, void* stream) {
     if (!a->workspace || a->workspace_bytes < dz_latent_attention_workspace_bytes(a->rows, a->heads, a->rank, a->splits))
       return DZ_ERR_WORKSPACE;
     p.tickets = (int*)a->workspace;
-    p.partial = (float*)((uint8_t*)a->workspace + latent_ticket_bytes(a->rows, a->heads));
+    p.partial = (float*)((uint8_t*)a->workspace + kTicketBytes);
+    if ((int64_t)a->rows * head_groups(a->heads) > kMaxTickets) return DZ_ERR_TOO_LARGE;
   }
   DZ_DISPATCH16(a->dtype, return head_tiles(a->heads) == 1 ? run_latent<T, 1>(p, st) : run_latent<T, 2>(p, st));
   return DZ_OK;

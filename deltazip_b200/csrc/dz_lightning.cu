@@ -544,8 +544,6 @@ int run_norm(const LightningParams& p, const I* o, int rows, cudaStream_t st) {
   return DZ_OK;
 }
 
-size_t ticket_bytes(int num_seqs) { return ((size_t)num_seqs * 4 + 255) & ~(size_t)255; }
-
 }  // namespace
 }  // namespace dz
 
@@ -562,7 +560,7 @@ int dz_lightning_chunk_supported(int dim, int vdim, int dtype) {
 
 size_t dz_lightning_workspace_bytes(int rows, int num_seqs, int heads, int vdim, int chunkwise) {
   if (rows <= 0 || num_seqs <= 0 || heads <= 0 || vdim <= 0 || chunkwise) return 0;
-  return ticket_bytes(num_seqs) + (size_t)rows * heads * vdim * 4;
+  return kTicketBytes + (size_t)rows * heads * vdim * 4;
 }
 
 int dz_lightning(const dz_lightning_args* a, void* stream) {
@@ -584,7 +582,7 @@ int dz_lightning(const dz_lightning_args* a, void* stream) {
       return DZ_ERR_WORKSPACE;
     const bool fused = a->rows == a->num_seqs;     // one token each: the norm rides on the last CTA of a row
     if (fused) p.tickets = (int*)a->workspace;
-    p.o = (float*)((uint8_t*)a->workspace + ticket_bytes(a->num_seqs));
+    p.o = (float*)((uint8_t*)a->workspace + kTicketBytes);
     int rc = DZ_OK;
     DZ_DISPATCH(a->dtype, rc = run_recurrent<T>(p, a->num_seqs, st));
     if (rc || fused) return rc;

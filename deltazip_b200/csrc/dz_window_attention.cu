@@ -644,9 +644,6 @@ int decode_grid_x(int heads, int kv_heads) {
   const int r = heads / kv_heads, g = decode_group(heads, kv_heads);
   return kv_heads * ((r + g - 1) / g);
 }
-size_t ticket_bytes(int num_seqs, int heads, int kv_heads) {
-  return (((size_t)num_seqs * decode_grid_x(heads, kv_heads) * 4) + 255) & ~(size_t)255;
-}
 
 // The 16-byte copies of the fast kernels need 8-element rows everywhere.
 bool fast_shapes(const AttnParams& p, int dtype) {
@@ -701,7 +698,7 @@ int dz_kv_append(const void* qkv, int64_t row_stride, int k_off, int k_width, in
 size_t dz_window_attention_workspace_bytes(int num_seqs, int heads, int kv_heads, int vdim, int splits) {
   if (num_seqs <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || vdim <= 0) return 0;
   if (splits <= 1) return kAttnStatusBytes;
-  return kAttnStatusBytes + ticket_bytes(num_seqs, heads, kv_heads) + (size_t)num_seqs * heads * splits * (vdim + 2) * 4;
+  return kAttnStatusBytes + kTicketBytes + (size_t)num_seqs * heads * splits * (vdim + 2) * 4;
 }
 
 int dz_window_attention(const dz_window_attention_args* a, void* stream) {
@@ -735,7 +732,8 @@ int dz_window_attention(const dz_window_attention_args* a, void* stream) {
                                                                                     a->vdim, a->splits))
         return DZ_ERR_WORKSPACE;
       tickets = (int*)((uint8_t*)a->workspace + kAttnStatusBytes);
-      partial = (float*)((uint8_t*)tickets + ticket_bytes(a->num_seqs, a->heads, a->kv_heads));
+      partial = (float*)((uint8_t*)tickets + kTicketBytes);
+      if ((int64_t)a->num_seqs * decode_grid_x(a->heads, a->kv_heads) > kMaxTickets) return DZ_ERR_TOO_LARGE;
     }
     const dim3 grid(decode_grid_x(a->heads, a->kv_heads), a->num_seqs, a->splits);
     const int g = decode_group(a->heads, a->kv_heads);

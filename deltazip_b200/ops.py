@@ -857,6 +857,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         splits = 1
     elif splits <= 0:
         splits = _balanced_splits(ctas, min(16, -(-block_tables.shape[1] * block_size // 256)))
+        splits = splits if ctas <= 65536 else 1
     out = torch.empty((rows, heads, rank), dtype=q.dtype, device=q.device)
     ws = _zeroed_scratch("latent_attention", q.device, lib().dz_latent_attention_workspace_bytes(rows, heads, rank, splits))
     args = _lib.LatentAttentionArgs(

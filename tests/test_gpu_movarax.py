@@ -174,6 +174,26 @@ def test_latent_attention_far_key_and_sink(dtype):
             assert np.abs(got[:far, 0, 1:]).max() < 0.5
 
 
+def test_split_launches_of_changing_batch_size_share_a_workspace():
+    """Large, small, large: what a launch keeps in the workspace is not where a larger one looks for its tickets."""
+    from deltazip_b200 import ops
+    g = torch.Generator(device="cuda").manual_seed(0)
+    rnd = lambda *s: torch.randn(s, generator=g, device="cuda").to(BF16)
+    t, bs, most = 200, 8, 96
+    table, q1 = i32(np.arange(25)[None].repeat(most, 0)), torch.arange(most + 1, dtype=torch.int32, device="cuda")
+    ctx = i32([t - 1] * most)
+    lat, ql = rnd(200, 1, 48), rnd(most, 4, 48)
+    k, v, x = rnd(200, 2, 128), rnd(200, 2, 128), rnd(most, 8 * 128)
+    calls = {"latent": lambda n, s: ops.latent_attention(ql[:n], lat, table[:n], q1[:n + 1], ctx[:n], 32, bs, 0.2, None, s),
+             "window": lambda n, s: ops.window_attention(x[:n], k, v, table[:n], q1[:n + 1], ctx[:n], 1, True, 4, bs, 0.1, 0,
+                                                         None, s),
+             "paged": lambda n, s: ops.paged_attention_decode(x[:n], k, v, table[:n], ctx[:n] + 1, 4, 2, bs, 0.1, s)}
+    for name, call in calls.items():
+        want = call(most, 1)
+        for n in (most, 1, most, 2, 3, most):
+            assert rel(host(call(n, 4)), host(want[:n])) < 1e-2, (name, n)
+
+
 def test_first_tokens_see_themselves_and_the_sink():
     r = LatentRun(2, 16, 8, 4, F32, sink=[0.4, -1.0])
     s = (host(r.q)[0] @ host(r.rows)[0]) * r.scale
