@@ -104,7 +104,7 @@ class LatentAttentionArgs(Structure):
         ("block_size", c_int32), ("q_starts", c_void_p), ("ctx_lens", c_void_p), ("num_seqs", c_int32),
         ("rows", c_int32), ("heads", c_int32), ("rank", c_int32), ("rot", c_int32), ("scale", c_float),
         ("sink", c_void_p), ("out", c_void_p), ("splits", c_int32), ("workspace", c_void_p),
-        ("workspace_bytes", c_size_t), ("dtype", c_int32),
+        ("workspace_bytes", c_size_t), ("dtype", c_int32), ("cache_rows", c_int64), ("status", c_void_p),
     ]
 
 

@@ -14,6 +14,7 @@
 // Neighbouring components (2i, 2i + 1) are rotated by position * freq[i]; the angle is formed and brought
 // into one turn in 64 bits, sine and cosine are 32-bit.  Scores, softmax weights and sums are 32-bit; a
 // weight enters its product as a hi + lo pair of 16-bit numbers.
+#include "dz_latent.cuh"
 #include "dz_window_attention.cuh"
 
 namespace dz {
@@ -67,8 +68,9 @@ struct RowParams {
   const long long* slots;
 };
 
-// grid (rows, 2): y = 0 the queries' rotation, y = 1 the latent's norm, its rotation and the cache append
-template <typename T, bool PAIRS>
+// The queries' rotation, and the latent's norm, its rotation and the cache append; a CTA per row.  VEC: the
+// parts consist of whole vectors of eight.
+template <typename T, bool PAIRS, bool VEC>
 __global__ void __launch_bounds__(kRowThreads)
 latent_rows_kernel(RowParams p) {
   extern __shared__ float2 s_cs[];
@@ -76,8 +78,7 @@ latent_rows_kernel(RowParams p) {
   pdl_wait();
   pdl_launch();
   const size_t row = blockIdx.x;
-  const long long slot = blockIdx.y ? p.slots[row] : 0;
-  if (slot < 0) return;
+  const long long slot = p.l_off >= 0 ? p.slots[row] : -1;
   const int half = p.rot / 2;
   const double pos = (double)p.positions[row];
   for (int i = threadIdx.x; i < half; i += kRowThreads) {
@@ -88,27 +89,66 @@ latent_rows_kernel(RowParams p) {
     sincosf((float)a, &s, &c);
     s_cs[i] = make_float2(c, s);
   }
-  __syncthreads();
   const T* x = (const T*)p.x + row * p.row_stride;
-  if (blockIdx.y == 0) {
+  const T* lat = x + p.l_off;
+  T* dst = (T*)p.cache + (size_t)slot * (p.rank + p.rot);
+  float ss = 0.f;
+  if (slot >= 0) {
+    if constexpr (VEC) {
+      for (int i = threadIdx.x * 8; i < p.rank; i += kRowThreads * 8) {
+        float f[8];
+        load8<T>(lat + i, f);
+#pragma unroll
+        for (int q = 0; q < 8; ++q) ss += f[q] * f[q];
+      }
+    } else {
+      for (int i = threadIdx.x; i < p.rank; i += kRowThreads) {
+        const float f = Cvt<T>::one(lat[i]);
+        ss += f * f;
+      }
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)p.rank + p.eps);        // also orders s_cs
+  if constexpr (VEC) {
+    const int per = p.rot / 8;
+    for (int j = threadIdx.x; j < p.heads * per; j += kRowThreads) {
+      const int head = j / per, i = (j - head * per) * 8;
+      const T* src = x + (size_t)head * (p.dim + p.rot) + p.dim + i;
+      T* to = p.q_out ? (T*)p.q_out + (row * p.heads + head) * (p.rank + p.rot) + p.rank + i : const_cast<T*>(src);
+      float f[8];
+      load8<T>(src, f);
+#pragma unroll
+      for (int q = 0; q < 8; q += 2) {
+        const float2 cs = s_cs[(i + q) / 2];
+        const float u = f[q], v = f[q + 1];
+        f[q] = u * cs.x - v * cs.y;
+        f[q + 1] = v * cs.x + u * cs.y;
+      }
+      store8<T>(to, f);
+    }
+  } else {
     for (int j = threadIdx.x; j < p.heads * half; j += kRowThreads) {
       const int head = j / half, i = j - head * half;
       const T* src = x + (size_t)head * (p.dim + p.rot) + p.dim + 2 * i;
-      T* dst = p.q_out ? (T*)p.q_out + (row * p.heads + head) * (p.rank + p.rot) + p.rank + 2 * i : const_cast<T*>(src);
-      rotate<T, PAIRS>(src, dst, s_cs[i]);
+      T* to = p.q_out ? (T*)p.q_out + (row * p.heads + head) * (p.rank + p.rot) + p.rank + 2 * i : const_cast<T*>(src);
+      rotate<T, PAIRS>(src, to, s_cs[i]);
     }
-    return;
   }
-  x += p.l_off;
-  T* dst = (T*)p.cache + (size_t)slot * (p.rank + p.rot);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < p.rank; i += kRowThreads) {
-    const float f = Cvt<T>::one(x[i]);
-    ss += f * f;
+  if (slot < 0) return;
+  if constexpr (VEC) {
+    for (int i = threadIdx.x * 8; i < p.rank; i += kRowThreads * 8) {
+      float f[8], w[8];
+      load8<T>(lat + i, f);
+      load8<float>(p.norm_w + i, w);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) f[q] = f[q] * inv * w[q];
+      store8<T>(dst + i, f);
+    }
+  } else {
+    for (int i = threadIdx.x; i < p.rank; i += kRowThreads) dst[i] = Cvt<T>::from(Cvt<T>::one(lat[i]) * inv * p.norm_w[i]);
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, s_part) / (float)p.rank + p.eps);
-  for (int i = threadIdx.x; i < p.rank; i += kRowThreads) dst[i] = Cvt<T>::from(Cvt<T>::one(x[i]) * inv * p.norm_w[i]);
-  for (int i = threadIdx.x; i < half; i += kRowThreads) rotate<T, PAIRS>(x + p.rank + 2 * i, dst + p.rank + 2 * i, s_cs[i]);
+  for (int i = threadIdx.x; i < half; i += kRowThreads)
+    rotate<T, PAIRS>(lat + p.rank + 2 * i, dst + p.rank + 2 * i, s_cs[i]);
 }
 
 // Cached rows of positions 0, 1, ... of every sequence into consecutive rows; grid (positions / 8, sequences).
@@ -129,29 +169,14 @@ latent_gather_kernel(const V* __restrict__ cache, const int* __restrict__ tables
 }
 
 // -------------------------------------------------------------------------------------------------
-// All heads of a row against the cached rows, 16-bit.  A CTA takes 16 MT heads (the MMA's M) of one row
+// All heads of a row against the cached rows, 16-bit, on warp MMAs: for what dz_latent_tc.cu does not take
+// (pages that are not a multiple of eight tokens).  A CTA takes 16 MT heads (the MMA's M) of one row
 // and a share of the keys, 64 per step, double-buffered through cp.async.  Eight warps: for the scores
 // (16 keys) x (half of the row's columns), for the sums a share of the latent's columns.  Grid (head
-// groups, rows, splits); with splits the last CTA of a (row, head group) to arrive at its ticket merges.
+// groups, rows, splits).
 // -------------------------------------------------------------------------------------------------
 constexpr int kKeys = 64, kLatentThreads = 256, kMaxGroups = 4;      // 16-column groups of the latent per warp
 constexpr int kLdS = kKeys + 4, kLdP = kKeys + 8;
-
-struct LatentParams {
-  const void* q;                         // [rows, heads, rank + rot]
-  const void* cache;                     // [slots, rank + rot]
-  const int* tables;
-  int table_width, block_size;
-  const int* q_starts;
-  const int* ctx_lens;
-  int num_seqs, rows, heads, rank, rot;
-  float scale;
-  const float* sink;
-  void* out;                             // [rows, heads, rank]
-  int splits;
-  float* partial;                        // [rows, heads, splits, rank + 2]
-  int* tickets;                          // [rows, head groups]
-};
 
 template <typename T, int MT>
 __global__ void __launch_bounds__(kLatentThreads, 1)
@@ -182,8 +207,8 @@ latent_decode_kernel(LatentParams p) {
     q0 = p.q_starts[seq];
   }
   const int n = p.ctx_lens[seq] + row - q0 + 1;                      // keys up to and with the row's own
-  const int per = (n + p.splits - 1) / p.splits;
-  const int t0 = split * per, t1 = min(n, t0 + per);
+  const int per = keys_per_split(n, p.splits);
+  const int t0 = min(n, split * per), t1 = min(n, t0 + per);
   const int* table = p.tables + (size_t)seq * p.table_width;
   const T* cache = (const T*)p.cache;
   const int chunks = d / 8;
@@ -370,37 +395,7 @@ latent_decode_kernel(LatentParams p) {
     pp[0] = s_m[tid];
     pp[1] = s_l[tid];
   }
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {
-    int* tk = p.tickets + (size_t)row * gridDim.x + blockIdx.x;
-    s_last = atomicAdd(tk, 1) == p.splits - 1;
-    if (s_last) *tk = 0;                                             // ready for the next launch
-  }
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
-  const int w = p.rank + 2;
-  for (int h = warp; h < live; h += 8) {                             // a warp merges a head
-    const size_t at = (size_t)row * p.heads + h0 + h;
-    const float* pp = p.partial + at * p.splits * w;
-    const float sk2 = p.sink ? p.sink[h0 + h] * kLog2e : -INFINITY;
-    float top = sk2;
-    for (int s = 0; s < p.splits; ++s) top = fmaxf(top, __ldcg(pp + s * w + p.rank));
-    float den = p.sink ? exp2f(sk2 - top) : 0.f;
-    for (int s = 0; s < p.splits; ++s) den += __ldcg(pp + s * w + p.rank + 1) * exp2f(__ldcg(pp + s * w + p.rank) - top);
-    const float inv = 1.f / den;
-    for (int c = lane * 2; c < p.rank; c += 64) {
-      float x = 0.f, y = 0.f;
-      for (int s = 0; s < p.splits; ++s) {
-        const float f = exp2f(__ldcg(pp + s * w + p.rank) - top);
-        const float2 v = __ldcg(reinterpret_cast<const float2*>(pp + s * w + c));
-        x += v.x * f;
-        y += v.y * f;
-      }
-      *reinterpret_cast<uint32_t*>((T*)p.out + at * p.rank + c) = Cvt<T>::down(x * inv, y * inv);
-    }
-  }
+  merge_splits<T>(p, row, h0, live, &s_last);
 }
 
 int head_tiles(int heads) { return heads <= 16 ? 1 : 2; }
@@ -444,9 +439,14 @@ int dz_latent_rows(const dz_latent_rows_args* a, void* stream) {
                  a->rank, a->norm_weight, a->eps, a->cache, (const long long*)a->slots};
   const bool pairs = a->dim % 2 == 0 && a->row_stride % 2 == 0 && ((a->q_out == nullptr && a->l_off < 0) || a->rank % 2 == 0) &&
                      (a->l_off < 0 || a->l_off % 2 == 0) && aligned16(a->x) && aligned16(a->q_out) && aligned16(a->cache);
-  const dim3 grid(a->rows, a->l_off >= 0 ? 2 : 1);
-  DZ_DISPATCH(a->dtype, DZ_CUDA_OK(launch_ex(pairs ? latent_rows_kernel<T, true> : latent_rows_kernel<T, false>, grid,
-                                             dim3(kRowThreads), (size_t)(a->rot / 2) * 8, 1, (cudaStream_t)stream, p)));
+  const bool vec = pairs && a->dim % 8 == 0 && a->rot % 8 == 0 && a->row_stride % 8 == 0 &&
+                   ((a->q_out == nullptr && a->l_off < 0) || a->rank % 8 == 0) &&
+                   (a->l_off < 0 || (a->l_off % 8 == 0 && aligned16(a->norm_weight)));
+  DZ_DISPATCH(a->dtype, DZ_CUDA_OK(launch_ex(vec     ? latent_rows_kernel<T, true, true>
+                                             : pairs ? latent_rows_kernel<T, true, false>
+                                                     : latent_rows_kernel<T, false, false>,
+                                             dim3(a->rows), dim3(kRowThreads), (size_t)(a->rot / 2) * 8, 1,
+                                             (cudaStream_t)stream, p)));
   return DZ_OK;
 }
 
@@ -513,7 +513,8 @@ int dz_latent_attention(const dz_latent_attention_args* a, void* stream) {
     return launch_attention_any(p, a->num_seqs, a->dtype, st);
   }
   LatentParams p = {a->q, a->cache, a->block_tables, a->table_width, a->block_size, a->q_starts, a->ctx_lens, a->num_seqs,
-                    a->rows, a->heads, a->rank, a->rot, a->scale, a->sink, a->out, a->splits, nullptr, nullptr};
+                    a->rows, a->heads, a->rank, a->rot, a->scale, a->sink, a->out, a->splits, nullptr, nullptr,
+                    a->cache_rows, a->status};
   if (a->splits > 1) {
     if (!a->workspace || a->workspace_bytes < dz_latent_attention_workspace_bytes(a->rows, a->heads, a->rank, a->splits))
       return DZ_ERR_WORKSPACE;
@@ -521,6 +522,7 @@ int dz_latent_attention(const dz_latent_attention_args* a, void* stream) {
     p.partial = (float*)((uint8_t*)a->workspace + kTicketBytes);
     if ((int64_t)a->rows * head_groups(a->heads) > kMaxTickets) return DZ_ERR_TOO_LARGE;
   }
+  if (latent_tc_supported(p, a->dtype)) return launch_latent_tc(p, a->dtype, st);
   DZ_DISPATCH16(a->dtype, return head_tiles(a->heads) == 1 ? run_latent<T, 1>(p, st) : run_latent<T, 2>(p, st));
   return DZ_OK;
 }

@@ -203,14 +203,14 @@ lightning_recurrent_kernel(LightningParams p, int vt) {
 // Chunkwise form, 16-bit activations.  Inside a chunk of L tokens, t = 0 ... L - 1,
 //   o_t = sum_{s <= t} w^(t-s) (q_t.k_s) v_s + w^(t+1) q_t S_start
 //   S_end = w^L S_start + sum_s w^(L-1-s) k_s v_s^T.
-// A CTA owns VT value columns of one (head, sequence) and walks the chunks.  Four warps bring a chunk in
+// A CTA owns VT value columns of one (head, sequence) and walks the chunks.  Eight warps bring a chunk in
 // while the one before is worked on: rows from memory, SiLU, rounded to 16 bits, v also times its power
-// of w.  Eight warps multiply; their slice of S stays in registers in 32 bits as accumulators of the
+// of w.  Eight others multiply; their slice of S stays in registers in 32 bits as accumulators of the
 // update.  32-bit operands (S, weighted scores, weighted v) enter the MMAs as hi + lo pairs.  A warp owns
 // NTW groups of eight of k's columns (64 NTW >= dim).  Writes o before the norm.  Grid (tiles of VT
 // columns, heads, sequences).
 // -------------------------------------------------------------------------------------------------
-constexpr int kMmaThreads = 256, kLoadThreads = 128, kChunkThreads = kMmaThreads + kLoadThreads;
+constexpr int kMmaThreads = 256, kLoadThreads = 256, kChunkThreads = kMmaThreads + kLoadThreads;
 
 __device__ __forceinline__ void bar_sync(int id, int count) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(count) : "memory"); }
 __device__ __forceinline__ void bar_arrive(int id, int count) {

@@ -4,7 +4,8 @@
 // The GEMM on tcgen05: 128 rows of an expert's matrix are the MMA's M, up to 256 of its entries the N, so a
 // decode batch (a few rows per expert) and a prompt batch take the same kernel with different tile widths.
 // Tiles (expert, rows of the matrix, entries) are dealt round-robin to one persistent CTA per SM, entries
-// first, so that the CTAs running at a time share matrix tiles in L2.  Roles: a TMA thread (matrix tile and
+// first, so that the CTAs running at a time share matrix tiles in L2; an expert's entries are cut into tiles
+// of equal width.  Roles: a TMA thread (matrix tile and
 // entry tile per 64-wide k step into a ring), an MMA thread (two TMEM accumulators), four epilogue warps
 // (scale, activation, store) that drain one accumulator while the next tile fills the other.  Tiles may run
 // past an expert's rows or entries: what is computed there is not stored.  All waits are bounded.
@@ -220,6 +221,8 @@ moe_gemm_any_kernel(MoeParams p) {
 constexpr int kMoeThreads = 192, kMaxStages = 10, kMaxExperts = 1024;    // warp 0 TMA, 1 MMA + TMEM, 2..5 epilogue
 constexpr int kWTile = 128 * 128;                                         // bytes of 128 matrix rows x 64 k
 
+constexpr int kXBox = 64;                                                 // entries per copy
+
 struct Tile { int e, row, count, n0; };
 
 template <typename T, int ACT>
@@ -289,9 +292,10 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
       const int mid = (lo + hi) >> 1;
       if (s_first[mid] <= vt) lo = mid; else hi = mid;
     }
+    // as few tiles as hold the expert's entries, of equal width
     const int rows = s_off[lo + 1] - s_off[lo], across = (rows + p.nt - 1) / p.nt, i = vt - s_first[lo];
-    const int t = i % across;
-    return Tile{lo, s_off[lo] + t * p.nt, min(p.nt, rows - t * p.nt), i / across * 128};
+    const int t = i % across, width = ((rows + across - 1) / across + 15) / 16 * 16;
+    return Tile{lo, s_off[lo] + t * width, min(width, rows - t * width), i / across * 128};
   };
 
   if (warp == 0) {
@@ -299,13 +303,14 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
       Ring r(p.stages, 1);
       for (int vt = blockIdx.x; vt < total; vt += gridDim.x) {
         const Tile t = tile(vt);
-        const int wrow = t.e * p.N + t.n0;
+        const int wrow = t.e * p.N + t.n0, box = min(kXBox, p.nt), boxes = (t.count + box - 1) / box;
         for (int ks = 0; ks < ksteps; ++ks) {
           mbar_wait(smem_u32(&s_empty[r.idx]), r.par, abort_flag, p.status);
           const uint32_t full = smem_u32(&s_full[r.idx]);
-          mbar_expect_tx(full, kWTile + x_bytes);
+          mbar_expect_tx(full, kWTile + boxes * box * 128);
           tma_load_2d(s_w + r.idx * kWTile, &map_w, ks * kBlockK, wrow, full);
-          tma_load_2d(s_x + r.idx * x_bytes, &map_x, ks * kBlockK, t.row, full);
+          for (int b = 0; b < boxes; ++b)
+            tma_load_2d(s_x + r.idx * x_bytes + b * box * 128, &map_x, ks * kBlockK, t.row + b * box, full);
           r.advance();
         }
       }
@@ -313,10 +318,10 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
   } else if (warp == 1) {
     if (lane == 0) {
       Ring r(p.stages, 0);
-      const uint32_t idesc = make_idesc<DT>(p.nt, false);
       int it = 0;
       for (int vt = blockIdx.x; vt < total; vt += gridDim.x, ++it) {
         const int a = it & 1;
+        const uint32_t idesc = make_idesc<DT>((tile(vt).count + 15) / 16 * 16, false);
         mbar_wait(smem_u32(&s_acc_empty[a]), ((it >> 1) & 1) ^ 1, abort_flag, p.status);
         tc_fence_after();
         for (int ks = 0; ks < ksteps; ++ks) {
@@ -389,7 +394,7 @@ int run_tc(MoeParams p, int typical, cudaStream_t st) {
   p.tmem_cols = std::max(32, 2 * p.nt);
   CUtensorMap map_w, map_x;
   int rc = make_map(&map_w, p.weights, p.experts * p.N, p.K, 128, kDt);
-  if (!rc) rc = make_map(&map_x, p.x, p.rows, p.K, p.nt, kDt);
+  if (!rc) rc = make_map(&map_x, p.x, p.rows, p.K, std::min(p.nt, kXBox), kDt);
   if (rc) return rc;
   int dev = 0, sms = 0;
   DZ_CUDA_OK(cudaGetDevice(&dev));

@@ -250,6 +250,54 @@ __device__ __forceinline__ void named_bar_sync(int id, int count) {
 }
 
 
+// An operand that lies [k][m or n] ("MN-major", v in o = p v): 64 columns (128 bytes) per slab, slabs
+// `lead` bytes apart, groups of eight rows 1024 bytes apart.
+__device__ __forceinline__ uint32_t desc_lo_mn(uint32_t saddr, int lead) {
+  return ((saddr >> 4) & 0x3FFFu) | ((uint32_t)(lead >> 4) << 16);
+}
+// One dense MMA, both operands in shared memory.
+__device__ __forceinline__ void umma_ss(uint32_t d, uint32_t a_lo, uint32_t b_lo, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t.reg .b64 da, db;\n\t"
+      "setp.ne.b32 p, %5, 0;\n\t"
+      "mov.b64 da, {%1, %3};\n\tmov.b64 db, {%2, %3};\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %4, p;\n\t}" ::"r"(d),
+      "r"(a_lo), "r"(b_lo), "r"(kDescHi), "r"(idesc), "r"(acc)
+      : "memory");
+}
+__device__ __forceinline__ void tmem_ld32(uint32_t a, float* f) {
+  uint32_t* v = reinterpret_cast<uint32_t*>(f);
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
+      "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
+        "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
+        "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
+        "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+      : "r"(a)
+      : "memory");
+}
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// byte offset of 16-byte chunk c of row r in a run of 64-element slabs of `slab` bytes
+__device__ __forceinline__ uint32_t swizzled(int r, int c, int slab) {
+  return (uint32_t)((c >> 3) * slab + r * 128 + (((c & 7) ^ (r & 7)) << 4));
+}
+
+// Bounded wait that polls (each try suspends for a while by itself) before it falls back to sleeping.
+__device__ __forceinline__ void bar_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int* status) {
+#pragma unroll 1
+  for (int i = 0; i < 32; ++i)
+    if (mbar_try_wait(smem_u32(bar), parity)) return;
+  mbar_wait_slow(smem_u32(bar), parity, abort_flag, status);
+}
+
 // position and wait parity inside a ring of `size` mbarrier-guarded slots
 struct Ring {
   int idx, par, size;

@@ -175,14 +175,14 @@ def _workspace(device, nbytes: int) -> torch.Tensor:
 
 
 def read_status(device=None) -> int:
-    """Reads and clears the status words the SBMM, window attention and expert kernels leave in the
+    """Reads and clears the status words the SBMM, window attention, latent attention and expert kernels leave in the
     current stream's workspaces (0 = ok, DZ_ERR_TIMEOUT = a bounded device-side wait ran
     out, DZ_ERR_INVALID_ARG = a wrong `tokens_sorted` promise).  Synchronises."""
     device = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
     found = 0
     for ws in (_workspaces.get((device.index, _stream())),
                _scratch.get(("window_attention", device.index, _stream())),
-               _scratch.get(("moe", device.index, _stream()))):
+               _scratch.get(("status", device.index, _stream()))):
         if ws is not None:
             host = ctypes.c_int(0)
             check(lib().dz_read_status(ws.data_ptr(), _stream(), ctypes.byref(host)), "dz_read_status")
@@ -864,7 +864,8 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         q=q.data_ptr(), cache=cache.data_ptr(), block_tables=block_tables.data_ptr(), table_width=block_tables.shape[1],
         block_size=block_size, q_starts=q_starts.data_ptr(), ctx_lens=ctx_lens.data_ptr(), num_seqs=ctx_lens.shape[0],
         rows=rows, heads=heads, rank=rank, rot=size - rank, scale=float(scale), sink=_ptr(sink), out=out.data_ptr(),
-        splits=splits, workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=code)
+        splits=splits, workspace=_ptr(ws), workspace_bytes=ws.numel() if ws is not None else 0, dtype=code,
+        cache_rows=cache.shape[0], status=_zeroed_scratch("status", q.device, 256).data_ptr())
     check(lib().dz_latent_attention(ctypes.byref(args), _stream()), "dz_latent_attention")
     return out
 
@@ -984,7 +985,7 @@ def moe_gemm(x: torch.Tensor, weights: torch.Tensor, offsets: torch.Tensor, scal
     if x.shape[1] != k or not x.is_contiguous() or not weights.is_contiguous() or x.dtype != weights.dtype:
         raise ValueError("x [rows, K] and weights [experts, N, K] must be contiguous and of one type")
     out = torch.empty((rows, n), dtype=x.dtype, device=x.device)
-    status = _zeroed_scratch("moe", x.device, 256)
+    status = _zeroed_scratch("status", x.device, 256)
     check(lib().dz_moe_gemm(x.data_ptr(), weights.data_ptr(), offsets.data_ptr(), _ptr(scale), out.data_ptr(), rows, n, k,
                             experts, ACTIVATIONS[activation] if activation else _lib.DZ_ACT_NONE, -(-rows // experts),
                             _any_dtype_code(x), status.data_ptr(), _stream()), "dz_moe_gemm")

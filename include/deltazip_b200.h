@@ -433,7 +433,9 @@ int dz_mlstm(const dz_mlstm_args* args, void* stream);
  *                     own position (which must be there already): softmax(q.[c|r] * scale, with one more
  *                     term exp(sink[head]) where sink is given) times c, [rows, heads, rank].  Row r of
  *                     sequence s has position ctx_lens[s] + r - q_starts[s].  With splits > 1 the
- *                     workspace must be zero-filled once before its first use
+ *                     workspace must be zero-filled once before its first use.  cache_rows: rows of the
+ *                     whole cache; status: a device word for a wait that ran out (may be NULL with
+ *                     cache_rows 0: then a kernel without such waits)
  */
 typedef struct dz_latent_rows_args {
   const void* x;
@@ -467,6 +469,8 @@ typedef struct dz_latent_attention_args {
   void* workspace;
   size_t workspace_bytes;
   int32_t dtype;
+  int64_t cache_rows;
+  int32_t* status;
 } dz_latent_attention_args;
 int dz_latent_attention_ctas(int rows, int heads, int rank, int rot, int dtype);
 size_t dz_latent_attention_workspace_bytes(int rows, int heads, int rank, int splits);
