@@ -385,17 +385,17 @@ latent_decode_kernel(LatentParams p) {
             if (p.splits == 1) {
               *reinterpret_cast<uint32_t*>((T*)p.out + at * p.rank + c) = Cvt<T>::down(x, y);
             } else {
-              *reinterpret_cast<float2*>(p.partial + (at * p.splits + split) * (p.rank + 2) + c) = make_float2(x, y);
+              *reinterpret_cast<float2*>(p.partial + (at * p.splits + split) * partial_row(p.rank) + c) = make_float2(x, y);
             }
           }
         }
   if (p.splits == 1) return;
   if (tid < live) {
-    float* pp = p.partial + (((size_t)row * p.heads + h0 + tid) * p.splits + split) * (p.rank + 2) + p.rank;
+    float* pp = p.partial + (((size_t)row * p.heads + h0 + tid) * p.splits + split) * partial_row(p.rank) + p.rank;
     pp[0] = s_m[tid];
     pp[1] = s_l[tid];
   }
-  merge_splits<T>(p, row, h0, live, &s_last);
+  merge_splits<T>(p, row, h0, live, &s_last, reinterpret_cast<float*>(smem_raw));
 }
 
 int head_tiles(int heads) { return heads <= 16 ? 1 : 2; }
@@ -478,7 +478,7 @@ int dz_latent_attention_ctas(int rows, int heads, int rank, int rot, int dtype) 
 
 size_t dz_latent_attention_workspace_bytes(int rows, int heads, int rank, int splits) {
   if (rows <= 0 || heads <= 0 || rank <= 0 || splits <= 1) return 0;
-  return kTicketBytes + (size_t)rows * heads * splits * (rank + 2) * 4;
+  return kTicketBytes + (size_t)rows * heads * splits * partial_row(rank) * 4;
 }
 
 int dz_latent_attention(const dz_latent_attention_args* a, void* stream) {

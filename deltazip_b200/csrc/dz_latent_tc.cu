@@ -5,14 +5,16 @@
 //   sums     O^T [latent, heads] += V^T P^T   V = the rows' first `rank` columns, read where they lie
 //                                             ("MN-major"), 128 of them per MMA tile
 //
-// With the heads along N the sums take a quarter of the tensor memory (32 columns per 128 of the latent)
-// and the MMAs are as long as there are heads.  The scores' M is 128 with the heads in the first lanes;
-// what the others hold comes from whatever lies behind Q and is never read.
+// With the heads along N the sums fit the tensor memory beside the scores and the MMAs are as long as there
+// are heads.  A weight is a hi + lo pair of 16-bit numbers; the his and the los are neighbouring columns of
+// one MMA, so that V is read once for both, and their sums are added at the end.  The scores' M is 128 with
+// the heads in the first lanes; what the others hold comes from whatever lies behind Q and is never read.
 //
-// Roles: warp 0 softmax (a lane owns a head: scores from TMEM, running maximum, exponentials, weights as
-// hi + lo 16-bit pairs into shared memory), warp 1 copies (TMA, one box per run of rows that lie together
-// in a page), warp 2 MMA issue, warp 3 tensor memory, warps 4-7 rescaling of the sums (rare: the maximum is
-// moved only when it has grown by more than 2^8) and the output.  All waits are bounded.
+// Roles: warps 0 and 4 softmax (a lane owns a head, a warp half of a tile's keys: scores from TMEM, running
+// maximum, exponentials, weights into shared memory), warps 1 and 3 copies (half of the columns each; TMA,
+// one box per slab and run of rows that lie together in a page), warp 2 MMA issue, warps 8-11 rescaling of
+// the sums (rare: the maximum is moved only when it has grown by more than 2^8) and the output.  All waits
+// are bounded.
 #include <algorithm>
 #include <numeric>
 
@@ -22,10 +24,10 @@
 namespace dz {
 namespace {
 
-constexpr int kTile = 64, kRing = 2, kTcThreads = 256, kTcHeads = 32, kMaxTiles = 4;   // tiles of 128 latent columns
+constexpr int kTile = 64, kRing = 2, kTcThreads = 384, kTcHeads = 32, kMaxTiles = 4;   // tiles of 128 latent columns
 constexpr int kSlabK = kTile * 128, kSlabH = kTcHeads * 128;                           // bytes: 64 keys, 32 heads x 64 columns
 constexpr float kGrowth = 8.f, kLog2 = 1.4426950408889634f;
-constexpr int kTmemCols = 256, kTmemO = 2 * kTile;                                     // S, S | O^T
+constexpr int kTmemCols = 512, kTmemO = 2 * kTile, kPairs = 2 * kTcHeads;              // S, S | O^T (hi | lo) per 128 of the latent
 
 template <typename T>
 __global__ void __launch_bounds__(kTcThreads, 1)
@@ -33,11 +35,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                         const LatentParams p, int run) {
   constexpr int DT = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
   extern __shared__ uint8_t smem_dyn[];
-  __shared__ uint64_t b_full[kRing], b_empty[kRing], b_s[2], b_dec[2], b_p[2], b_pv[2], b_o, b_q, b_tail;
-  __shared__ float s_f[kTcHeads], s_out[kTcHeads];
+  __shared__ uint64_t b_full[kRing][2], b_empty[kRing], b_s[2], b_dec[2], b_p[2], b_pv[2], b_o, b_q, b_tail[2];
+  __shared__ float s_f[kTcHeads], s_out[kTcHeads], s_top[2][2][kTcHeads], s_sum[kTcHeads];
   __shared__ int s_need[2], s_seq, s_abort, s_last;
   __shared__ uint32_t s_tmem;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
   const int h0 = blockIdx.x * kTcHeads, row = blockIdx.y, split = blockIdx.z, live = min(kTcHeads, p.heads - h0);
   const int d = p.rank + p.rot, slabs = (d + 63) / 64, tiles_m = (p.rank + 127) / 128;
   const int hn = p.heads <= 16 ? 16 : 32;                              // the MMAs' N
@@ -46,18 +48,20 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   volatile int* abort_flag = &s_abort;
   if (tid == 0) {
     for (int i = 0; i < kRing; ++i) {
-      mbar_init(smem_u32(&b_full[i]), 1);
+      mbar_init(smem_u32(&b_full[i][0]), 1);
+      mbar_init(smem_u32(&b_full[i][1]), 1);
       mbar_init(smem_u32(&b_empty[i]), 1);
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(smem_u32(&b_s[i]), 1);
-      mbar_init(smem_u32(&b_dec[i]), 1);
-      mbar_init(smem_u32(&b_p[i]), 5);
+      mbar_init(smem_u32(&b_dec[i]), 2);
+      mbar_init(smem_u32(&b_p[i]), 6);
       mbar_init(smem_u32(&b_pv[i]), 1);
     }
     mbar_init(smem_u32(&b_o), 1);
     mbar_init(smem_u32(&b_q), 1);
-    mbar_init(smem_u32(&b_tail), 1);
+    mbar_init(smem_u32(&b_tail[0]), 1);
+    mbar_init(smem_u32(&b_tail[1]), 1);
     s_abort = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     fence_proxy_async();
@@ -88,33 +92,34 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   tc_fence_after();
   const uint32_t tmem = s_tmem;
 
-  if (warp == 1) {
+  const int half = (slabs + 1) / 2;                                    // slabs of the first copy warp
+  if (warp == 1 || warp == 3) {
     // ---- copies ----
     const int* table = p.tables + (size_t)seq * p.table_width;
-    if (lane == 0 && tiles > 0) {
-      mbar_expect_tx(smem_u32(&b_q), slabs * hn * 128);
-      for (int i = 0; i < slabs; ++i) tma_load_2d(s_q + i * kSlabH, &map_q, i * 64, row * p.heads + h0, smem_u32(&b_q));
+    const int part = warp >> 1, c0 = part ? half : 0, c1 = part ? slabs : half;
+    if (tiles > 0 && part == 0) {
+      warp_mbar_expect_tx(smem_u32(&b_q), slabs * hn * 128);
+      for (int i = 0; i < slabs; ++i) warp_tma_load_2d(s_q + i * kSlabH, &map_q, i * 64, row * p.heads + h0, smem_u32(&b_q));
     }
     for (int j = 0; j < tiles; ++j) {
       const int st = j % kRing, base = t0 + j * kTile, valid = min(kTile, t1 - base);
-      const uint32_t dst = s_k + st * stage, full = smem_u32(&b_full[st]);
+      const uint32_t dst = s_k + st * stage, full = smem_u32(&b_full[st][part]);
       // the cache row of every run of rows of the tile, a lane each
       const int runs = (valid + run - 1) / run, t = base + lane * run;
       const int at = lane < runs ? table[t / p.block_size] * p.block_size + t % p.block_size : 0;
       bar_wait(&b_empty[st], ((j / kRing) & 1) ^ 1, abort_flag, p.status);
-      const bool tail = valid < kTile;
-      const uint32_t bar = tail ? smem_u32(&b_tail) : full;            // at most one tile of a CTA is cut
-      if (lane == 0) mbar_expect_tx(bar, runs * run * slabs * 128);
       __syncwarp();
-      for (int i = lane; i < ((runs * slabs + 31) & ~31); i += 32) {
-        const int r = i / slabs, c = i - r * slabs;
-        const int from = __shfl_sync(0xffffffffu, at, r & 31);
-        if (r < runs) tma_load_2d(dst + c * kSlabK + r * run * 128, &map_k, c * 64, from, bar);
+      const bool tail = valid < kTile;
+      const uint32_t bar = tail ? smem_u32(&b_tail[part]) : full;      // at most one tile of a CTA is cut
+      warp_mbar_expect_tx(bar, runs * run * (c1 - c0) * 128);
+      for (int r = 0; r < runs; ++r) {
+        const int from = __shfl_sync(0xffffffffu, at, r);
+        for (int c = c0; c < c1; ++c) warp_tma_load_2d(dst + c * kSlabK + r * run * 128, &map_k, c * 64, from, bar);
       }
       if (tail) {                                                      // rows past the end must not count: make them zero
-        bar_wait(&b_tail, 0, abort_flag, p.status);
+        bar_wait(&b_tail[part], 0, abort_flag, p.status);
         for (int i = valid * 8 + lane; i < kTile * 8; i += 32)
-          for (int c = 0; c < slabs; ++c) sts128(dst + c * kSlabK + i * 16, make_uint4(0, 0, 0, 0));
+          for (int c = c0; c < c1; ++c) sts128(dst + c * kSlabK + i * 16, make_uint4(0, 0, 0, 0));
         fence_proxy_async();
         __syncwarp();
         if (lane == 0) mbar_arrive(full);
@@ -122,65 +127,85 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     }
   } else if (warp == 2) {
     // ---- MMA issue ----
-    if (lane == 0 && tiles > 0) {
-      const uint32_t id_s = make_idesc<DT>(kTile, false), id_o = make_idesc<DT>(hn, false) | (1u << 15);   // A transposed
-      const int ksteps = (d + 15) / 16;
+    if (tiles > 0) {
+      const uint32_t id_s = make_idesc<DT>(kTile, false), id_o = make_idesc<DT>(2 * hn, false) | (1u << 15);   // A transposed
       auto scores = [&](int j) {
         const int st = j % kRing;
-        bar_wait(&b_full[st], (j / kRing) & 1, abort_flag, p.status);
-        tc_fence_after();
         const uint32_t a = desc_lo(s_q), b = desc_lo(s_k + st * stage);
-        for (int k = 0; k < ksteps; ++k) {
-          const uint32_t in = (uint32_t)((k & 3) * 2), slab = (uint32_t)(k >> 2);
-          umma_ss(tmem + (j & 1) * kTile, a + slab * (kSlabH >> 4) + in, b + slab * (kSlabK >> 4) + in, id_s, k > 0);
+        auto slab = [&](int c, int n) {                                // n MMAs of 16 columns
+          for (int k = 0; k < n; ++k)
+            warp_umma_ss(tmem + (j & 1) * kTile, a + c * (kSlabH >> 4) + k * 2, b + c * (kSlabK >> 4) + k * 2, id_s, c + k > 0);
+        };
+        for (int part = 0; part < 2; ++part) {
+          bar_wait(&b_full[st][part], (j / kRing) & 1, abort_flag, p.status);
+          __syncwarp();
+          tc_fence_after();
+          const int c1 = part ? slabs : half;
+          int c = part ? half : 0;
+          for (; c < min(c1, d / 64); ++c) slab(c, 4);
+          if (c < c1) slab(c, (d % 64 + 15) / 16);
         }
-        umma_commit(smem_u32(&b_s[j & 1]));
+        warp_umma_commit(smem_u32(&b_s[j & 1]));
       };
       bar_wait(&b_q, 0, abort_flag, p.status);
       scores(0);
       for (int j = 0; j < tiles; ++j) {
-        if (j + 1 < tiles) scores(j + 1);
         const int st = j % kRing, buf = j & 1;
-        bar_wait(&b_p[buf], (j >> 1) & 1, abort_flag, p.status);
-        tc_fence_after();
-        const uint32_t hi = desc_lo(s_p + buf * 2 * kSlabH), lo = desc_lo(s_p + (buf * 2 + 1) * kSlabH);
-        for (int m = 0; m < tiles_m; ++m) {
-          const uint32_t v = desc_lo_mn(s_k + st * stage + m * 2 * kSlabK, kSlabK), o = tmem + kTmemO + m * kTcHeads;
-#pragma unroll
-          for (int k = 0; k < kTile / 16; ++k) {                       // 16 keys: 2048 bytes of v, 32 of p
-            umma_ss(o, v + k * 128, hi + k * 2, id_o, (j > 0 || k > 0) ? 1u : 0u);
-            umma_ss(o, v + k * 128, lo + k * 2, id_o, 1u);
+        // the next tile's scores under this one's softmax, if it is here in time
+        bool ahead = j + 1 >= tiles;
+        for (int i = 0; i < 4096 && !ahead; ++i) {
+          if (__any_sync(0xffffffffu, mbar_test(smem_u32(&b_p[buf]), (j >> 1) & 1))) break;
+          if (__any_sync(0xffffffffu, mbar_test(smem_u32(&b_full[(j + 1) % kRing][0]), ((j + 1) / kRing) & 1) &&
+                                          mbar_test(smem_u32(&b_full[(j + 1) % kRing][1]), ((j + 1) / kRing) & 1))) {
+            scores(j + 1);
+            ahead = true;
           }
         }
-        umma_commit(smem_u32(&b_empty[st]));
-        umma_commit(smem_u32(&b_pv[buf]));
+        bar_wait(&b_p[buf], (j >> 1) & 1, abort_flag, p.status);
+        __syncwarp();
+        tc_fence_after();
+        const uint32_t w = desc_lo(s_p + buf * 2 * kSlabH);
+        for (int m = 0; m < tiles_m; ++m) {
+          const uint32_t v = desc_lo_mn(s_k + st * stage + m * 2 * kSlabK, kSlabK), o = tmem + kTmemO + m * kPairs;
+#pragma unroll
+          for (int k = 0; k < kTile / 16; ++k)                         // 16 keys: 2048 bytes of v, 32 of p
+            warp_umma_ss(o, v + k * 128, w + k * 2, id_o, (j > 0 || k > 0) ? 1u : 0u);
+        }
+        warp_umma_commit(smem_u32(&b_empty[st]));
+        warp_umma_commit(smem_u32(&b_pv[buf]));
+        if (!ahead) scores(j + 1);
       }
-      umma_commit(smem_u32(&b_o));
+      warp_umma_commit(smem_u32(&b_o));
     }
-  } else if (warp == 0) {
+  } else if (warp == 0 || warp == 4) {
     // ---- softmax ----
+    constexpr int kMine = kTile / 2;
+    const int part = warp >> 2;
     const float scale2 = p.scale * kLog2;
     float m = -INFINITY, l = 0.f;
     for (int j = 0; j < tiles; ++j) {
-      const int buf = j & 1, valid = min(kTile, t1 - t0 - j * kTile);
+      const int buf = j & 1, valid = min(kTile, t1 - t0 - j * kTile) - part * kMine;
       bar_wait(&b_s[buf], (j >> 1) & 1, abort_flag, p.status);
+      __syncwarp();
       tc_fence_after();
-      float s[kTile];
-      tmem_ld32(tmem + buf * kTile, s);
-      tmem_ld32(tmem + buf * kTile + 32, s + 32);
+      float s[kMine];
+      tmem_ld32(tmem + buf * kTile + part * kMine, s);
       tmem_wait_ld();
       if (lane >= live) {                                              // lanes without a head
 #pragma unroll
-        for (int c = 0; c < kTile; ++c) s[c] = 0.f;
+        for (int c = 0; c < kMine; ++c) s[c] = 0.f;
       }
-      if (valid < kTile) {
+      if (valid < kMine) {
 #pragma unroll
-        for (int c = 0; c < kTile; ++c) s[c] = c < valid ? s[c] : -INFINITY;
+        for (int c = 0; c < kMine; ++c) s[c] = c < valid ? s[c] : -INFINITY;
       }
       float mx[4] = {s[0], s[1], s[2], s[3]};
 #pragma unroll
-      for (int c = 4; c < kTile; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
-      const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale2;
+      for (int c = 4; c < kMine; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
+      float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+      s_top[buf][part][lane] = top;
+      named_bar_sync(1, 64);
+      top = fmaxf(top, s_top[buf][part ^ 1][lane]) * scale2;           // the tile's first key is there: finite
       float f = 1.f;
       if (j == 0) {
         m = top;
@@ -189,12 +214,12 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         m = top;
         l *= f;
       }
-      const bool need = __any_sync(0xffffffffu, f != 1.f);
+      const bool need = __any_sync(0xffffffffu, f != 1.f);             // the same in both warps
       if (j >= 2) bar_wait(&b_pv[buf], ((j >> 1) - 1) & 1, abort_flag, p.status);       // these weights have been used
-      const uint32_t ph = s_p + buf * 2 * kSlabH, pl = ph + kSlabH;
+      const uint32_t ph = s_p + buf * 2 * kSlabH, pl = ph + hn * 128;
       float sum[2] = {0.f, 0.f};
 #pragma unroll
-      for (int c = 0; c < kTile / 8; ++c) {
+      for (int c = 0; c < kMine / 8; ++c) {
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
@@ -203,13 +228,17 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
           sum[1] += b;
           split_pair<T>(a, b, hi[i], lo[i]);
         }
-        const uint32_t at = swizzled(lane, c, kSlabH);
-        sts128(ph + at, make_uint4(hi[0], hi[1], hi[2], hi[3]));
-        sts128(pl + at, make_uint4(lo[0], lo[1], lo[2], lo[3]));
+        if (lane < hn) {
+          const uint32_t at = swizzled(lane, part * (kMine / 8) + c, kSlabH);
+          sts128(ph + at, make_uint4(hi[0], hi[1], hi[2], hi[3]));
+          sts128(pl + at, make_uint4(lo[0], lo[1], lo[2], lo[3]));
+        }
       }
       l += sum[0] + sum[1];
-      s_f[lane] = f;
-      if (lane == 0) s_need[buf] = need;
+      if (part == 0) {
+        s_f[lane] = f;
+        if (lane == 0) s_need[buf] = need;
+      }
       fence_proxy_async();
       tc_fence_before();
       __syncwarp();
@@ -219,19 +248,22 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       }
       if (need) bar_wait(&b_p[buf], (j >> 1) & 1, abort_flag, p.status);                // s_f is written again next
     }
-    if (lane < live) {
+    if (part == 1) s_sum[lane] = l;
+    named_bar_sync(1, 64);
+    if (part == 0 && lane < live) {
+      l += s_sum[lane];
       float f = 1.f;
       if (p.splits == 1) {
         const float sk2 = p.sink ? p.sink[h0 + lane] * kLog2 : -INFINITY, top = fmaxf(m, sk2), c = exp2f(m - top);
         f = c / (l * c + exp2f(sk2 - top));
       } else {
-        float* pp = p.partial + (((size_t)row * p.heads + h0 + lane) * p.splits + split) * (p.rank + 2) + p.rank;
+        float* pp = p.partial + (((size_t)row * p.heads + h0 + lane) * p.splits + split) * partial_row(p.rank) + p.rank;
         pp[0] = m;
         pp[1] = l;
       }
       s_out[lane] = f;
     }
-  } else if (warp >= 4) {
+  } else if (warp >= 8) {
     // ---- rescaling ----
     const uint32_t t_o = tmem + kTmemO + ((uint32_t)((warp & 3) * 32) << 16);
     for (int j = 0; j < tiles; ++j) {
@@ -240,15 +272,16 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       if (s_need[buf]) {                                               // never the first tile
         bar_wait(&b_pv[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag, p.status);         // O holds the products so far
         tc_fence_after();
-        for (int i = 0; i < tiles_m; ++i) {
-          float o[32];
-          tmem_ld32(t_o + i * kTcHeads, o);
-          tmem_wait_ld();
+        for (int i = 0; i < tiles_m * kPairs; i += kPairs)
+          for (int part = 0; part < 2 * hn; part += 32) {               // 32 columns: his, los, or 16 of each
+            float o[32];
+            tmem_ld32(t_o + i + part, o);
+            tmem_wait_ld();
 #pragma unroll
-          for (int c = 0; c < 32; ++c) o[c] *= s_f[c];
-          tmem_st16(t_o + i * kTcHeads, reinterpret_cast<const uint32_t*>(o));
-          tmem_st16(t_o + i * kTcHeads + 16, reinterpret_cast<const uint32_t*>(o + 16));
-        }
+            for (int c = 0; c < 32; ++c) o[c] *= s_f[c & (hn - 1)];
+            tmem_st16(t_o + i + part, reinterpret_cast<const uint32_t*>(o));
+            tmem_st16(t_o + i + part + 16, reinterpret_cast<const uint32_t*>(o + 16));
+          }
         tmem_wait_st();
         tc_fence_before();
       }
@@ -259,23 +292,29 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     tc_fence_after();
   }
   __syncthreads();
-  if (warp >= 4) {
+  if (warp >= 8) {
     // ---- output ----
+    // small loops: this code runs once, and fetching it costs more than running it
     const uint32_t t_o = tmem + kTmemO + ((uint32_t)((warp & 3) * 32) << 16);
+    const size_t at = (size_t)row * p.heads + h0;
+    const int step = p.splits == 1 ? p.rank : p.splits * partial_row(p.rank);        // from a head to the next
+#pragma unroll 1
     for (int i = 0; i < tiles_m; ++i) {
       const int c = i * 128 + (warp & 3) * 32 + lane;
-      float o[32];
-      if (tiles > 0) {
-        tmem_ld32(t_o + i * kTcHeads, o);
+      T* out = (T*)p.out + at * p.rank + c;
+      float* part = p.partial + (at * p.splits + split) * partial_row(p.rank) + c;
+#pragma unroll 1
+      for (int h = 0; h < live; h += 8) {
+        uint32_t hi[8], lo[8];
+        tmem_ld8(t_o + i * kPairs + h, hi);
+        tmem_ld8(t_o + i * kPairs + hn + h, lo);
         tmem_wait_ld();
-      }
-      if (c < p.rank) {
 #pragma unroll
-        for (int h = 0; h < kTcHeads; ++h) {
-          if (h < live) {
-            const size_t at = (size_t)row * p.heads + h0 + h;
-            if (p.splits == 1) ((T*)p.out)[at * p.rank + c] = Cvt<T>::from(o[h] * s_out[h]);
-            else p.partial[(at * p.splits + split) * (p.rank + 2) + c] = tiles > 0 ? o[h] : 0.f;
+        for (int e = 0; e < 8; ++e) {
+          const float o = tiles > 0 ? __uint_as_float(hi[e]) + __uint_as_float(lo[e]) : 0.f;
+          if (h + e < live && c < p.rank) {
+            if (p.splits == 1) out[(h + e) * step] = Cvt<T>::from(o * s_out[h + e]);
+            else part[(h + e) * step] = o;
           }
         }
       }
@@ -292,7 +331,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(kTmemCols) : "memory");
   }
-  if (p.splits > 1) merge_splits<T>(p, row, h0, live, &s_last);
+  if (p.splits > 1) merge_splits<T>(p, row, h0, live, &s_last, reinterpret_cast<float*>(smem_dyn));
 }
 
 size_t tc_smem(int d) {

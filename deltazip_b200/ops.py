@@ -18,6 +18,7 @@ one for thousands of prompt tokens.
 from __future__ import annotations
 
 import ctypes
+import functools
 from typing import NamedTuple, Optional, Tuple
 
 import torch
@@ -830,6 +831,7 @@ def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, block_size: i
     return out
 
 
+@functools.lru_cache(maxsize=4096)
 def _balanced_splits(ctas: int, most: int, sms: int = 148) -> int:
     """Splits of every CTA's work with the fullest last wave; fewer where that gains little."""
     best, score = 1, 0.0
