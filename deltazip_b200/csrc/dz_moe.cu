@@ -5,8 +5,8 @@
 // decode batch (a few rows per expert) and a prompt batch take the same kernel with different tile widths.
 // Tiles (expert, rows of the matrix, entries) are dealt round-robin to one persistent CTA per SM, entries
 // first, so that the CTAs running at a time share matrix tiles in L2; an expert's entries are cut into tiles
-// of equal width.  Roles: a TMA thread (matrix tile and
-// entry tile per 64-wide k step into a ring), an MMA thread (two TMEM accumulators), four epilogue warps
+// of equal width.  Roles: a TMA warp (matrix tile and
+// entry tile per 64-wide k step into a ring), an MMA warp (two TMEM accumulators), four epilogue warps
 // (scale, activation, store) that drain one accumulator while the next tile fills the other.  Tiles may run
 // past an expert's rows or entries: what is computed there is not stored.  All waits are bounded.
 #include <algorithm>
@@ -234,7 +234,7 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
   __shared__ int s_off[kMaxExperts + 1], s_first[kMaxExperts + 1];        // first row, first tile of every expert
   __shared__ int s_abort;
   __shared__ uint32_t s_tmem_base;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
   const uint32_t s_w = (smem_u32(smem_dyn) + 1023u) & ~1023u;
   const uint32_t x_bytes = p.nt * 128, s_x = s_w + p.stages * kWTile;
   if (threadIdx.x == 0) {
@@ -299,41 +299,40 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
   };
 
   if (warp == 0) {
-    if (lane == 0) {
-      Ring r(p.stages, 1);
-      for (int vt = blockIdx.x; vt < total; vt += gridDim.x) {
-        const Tile t = tile(vt);
-        const int wrow = t.e * p.N + t.n0, box = min(kXBox, p.nt), boxes = (t.count + box - 1) / box;
-        for (int ks = 0; ks < ksteps; ++ks) {
-          mbar_wait(smem_u32(&s_empty[r.idx]), r.par, abort_flag, p.status);
-          const uint32_t full = smem_u32(&s_full[r.idx]);
-          mbar_expect_tx(full, kWTile + boxes * box * 128);
-          tma_load_2d(s_w + r.idx * kWTile, &map_w, ks * kBlockK, wrow, full);
-          for (int b = 0; b < boxes; ++b)
-            tma_load_2d(s_x + r.idx * x_bytes + b * box * 128, &map_x, ks * kBlockK, t.row + b * box, full);
-          r.advance();
-        }
+    Ring r(p.stages, 1);
+    for (int vt = blockIdx.x; vt < total; vt += gridDim.x) {
+      const Tile t = tile(vt);
+      const int wrow = t.e * p.N + t.n0, box = min(kXBox, p.nt), boxes = (t.count + box - 1) / box;
+      for (int ks = 0; ks < ksteps; ++ks) {
+        mbar_wait(smem_u32(&s_empty[r.idx]), r.par, abort_flag, p.status);
+        __syncwarp();
+        const uint32_t full = smem_u32(&s_full[r.idx]);
+        warp_mbar_expect_tx(full, kWTile + boxes * box * 128);
+        warp_tma_load_2d(s_w + r.idx * kWTile, &map_w, ks * kBlockK, wrow, full);
+        for (int b = 0; b < boxes; ++b)
+          warp_tma_load_2d(s_x + r.idx * x_bytes + b * box * 128, &map_x, ks * kBlockK, t.row + b * box, full);
+        r.advance();
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
-      Ring r(p.stages, 0);
-      int it = 0;
-      for (int vt = blockIdx.x; vt < total; vt += gridDim.x, ++it) {
-        const int a = it & 1;
-        const uint32_t idesc = make_idesc<DT>((tile(vt).count + 15) / 16 * 16, false);
-        mbar_wait(smem_u32(&s_acc_empty[a]), ((it >> 1) & 1) ^ 1, abort_flag, p.status);
+    Ring r(p.stages, 0);
+    int it = 0;
+    for (int vt = blockIdx.x; vt < total; vt += gridDim.x, ++it) {
+      const int a = it & 1;
+      const uint32_t idesc = make_idesc<DT>((tile(vt).count + 15) / 16 * 16, false), acc = tmem_base + a * p.nt;
+      mbar_wait(smem_u32(&s_acc_empty[a]), ((it >> 1) & 1) ^ 1, abort_flag, p.status);
+      tc_fence_after();
+      for (int ks = 0; ks < ksteps; ++ks) {
+        mbar_wait(smem_u32(&s_full[r.idx]), r.par, abort_flag, p.status);
+        __syncwarp();
         tc_fence_after();
-        for (int ks = 0; ks < ksteps; ++ks) {
-          mbar_wait(smem_u32(&s_full[r.idx]), r.par, abort_flag, p.status);
-          tc_fence_after();
-          umma_ss_x4(tmem_base + a * p.nt, desc_lo(s_w + r.idx * kWTile), desc_lo(s_x + r.idx * x_bytes), idesc,
-                     ks > 0 ? 1u : 0u);
-          umma_commit(smem_u32(&s_empty[r.idx]));
-          r.advance();
-        }
-        umma_commit(smem_u32(&s_acc_full[a]));
+        const uint32_t w = desc_lo(s_w + r.idx * kWTile), x = desc_lo(s_x + r.idx * x_bytes);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) warp_umma_ss(acc, w + 2 * k, x + 2 * k, idesc, ks > 0 || k > 0);
+        warp_umma_commit(smem_u32(&s_empty[r.idx]));
+        r.advance();
       }
+      warp_umma_commit(smem_u32(&s_acc_full[a]));
     }
   } else {
     const int q = warp & 3;

@@ -74,15 +74,18 @@ __device__ __forceinline__ void cp_async16_u32(uint32_t dst, const void* src, bo
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
 }
 
-__device__ __forceinline__ void umma_ts(uint32_t d, uint32_t a, uint32_t b_lo, uint32_t idesc, uint32_t acc) {
+// As warp_umma_ss, with the first operand in tensor memory.
+__device__ __forceinline__ void warp_umma_ts(uint32_t d, uint32_t a, uint32_t b_lo, uint32_t idesc, uint32_t acc) {
   asm volatile(
-      "{\n\t.reg .pred p;\n\t.reg .b64 db;\n\t"
+      "{\n\t.reg .pred p, e;\n\t.reg .b64 db;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
       "setp.ne.b32 p, %5, 0;\n\t"
       "mov.b64 db, {%2, %3};\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], db, %4, p;\n\t}" ::"r"(d),
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], db, %4, p;\n\t}" ::"r"(d),
       "r"(a), "r"(b_lo), "r"(kDescHi), "r"(idesc), "r"(acc)
       : "memory");
 }
+
 template <typename T, int kStages>
 __global__ void __launch_bounds__(kThreadsTc, 1)
 window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
@@ -92,7 +95,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   __shared__ uint64_t b_full[kStages], b_empty[kStages], b_s[2][2], b_p[2][2], b_pv[2], b_o[2], b_q;
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
   const int seq = blockIdx.z, head = blockIdx.y % p.heads, v0 = (blockIdx.y / p.heads) * 128;
   pdl_wait();
   pdl_launch();
@@ -161,48 +164,54 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 
   if (warp >= 10) {
     // ---- MMA issue ----
-    if (lane == 0) {
-      const uint32_t id_s = make_idesc<DT>(kTileKeys, false);
-      const uint32_t id_o = make_idesc<DT>(vs * 64, false) | (1u << 16);       // B transposed
-      const uint32_t t_s = tmem + g * 128, t_o = tmem + 256 + g * 128;
-      const int ksteps = (p.dim + 15) / 16;
-      auto scores = [&](int j) {
-        const int st = j % kStages, buf = (j - ta) & 1;
-        bar_wait(&b_full[st], (j / kStages) & 1, abort_flag, p.status);
-        tc_fence_after();
-        const uint32_t a = desc_lo(s_q + g * ks * kSlabQ), b = desc_lo(s_k + st * ks * kSlab);
-        for (int k = 0; k < ksteps; ++k) {
-          const uint32_t in = (uint32_t)((k & 3) * 2), slab = (uint32_t)(k >> 2);
-          umma_ss(t_s + buf * 64, a + slab * (kSlabQ >> 4) + in, b + slab * (kSlab >> 4) + in, id_s, k > 0);
-        }
-        umma_commit(smem_u32(&b_s[g][buf]));
-      };
-      bar_wait(&b_q, 0, abort_flag, p.status);
-      for (int j = 0; j < tiles; ++j) {
-        const int st = j % kStages;
-        if (j < ta || j >= tb) {
-          bar_wait(&b_full[st], (j / kStages) & 1, abort_flag, p.status);
-          mbar_arrive(smem_u32(&b_empty[st]));
-          continue;
-        }
-        if (j == ta) {
-          scores(j);
-          if (j + 1 < tb) scores(j + 1);
-        }
-        const int n = j - ta, buf = n & 1;
-        bar_wait(&b_p[g][buf], (n >> 1) & 1, abort_flag, p.status);
-        tc_fence_after();
-        const uint32_t b = desc_lo_mn(s_v + st * vs * kSlab, kSlab), pw = t_s + buf * 64;
+    const uint32_t id_s = make_idesc<DT>(kTileKeys, false);
+    const uint32_t id_o = make_idesc<DT>(vs * 64, false) | (1u << 16);       // B transposed
+    const uint32_t t_s = tmem + g * 128, t_o = tmem + 256 + g * 128, s_qg = s_q + g * ks * kSlabQ;
+    const int rest = (p.dim % 64 + 15) / 16;                                 // MMAs of the last slab, 0: a whole one
+    auto scores = [&](int j) {
+      const int st = j % kStages, buf = (j - ta) & 1;
+      bar_wait(&b_full[st], (j / kStages) & 1, abort_flag, p.status);
+      __syncwarp();
+      tc_fence_after();
+      const uint32_t a = desc_lo(s_qg), b = desc_lo(s_k + st * ks * kSlab), d = t_s + buf * 64;
+      for (int c = 0; c < ks; ++c) {
+        const uint32_t ac = a + c * (kSlabQ >> 4), bc = b + c * (kSlab >> 4);
+        if (c + 1 < ks || rest == 0) {
 #pragma unroll
-        for (int k = 0; k < kTileKeys / 16; ++k) {                              // 16 keys: 2048 bytes of v
-          umma_ts(t_o, pw + k * 8, b + k * 128, id_o, (n > 0 || k > 0) ? 1u : 0u);
-          umma_ts(t_o, pw + 32 + k * 8, b + k * 128, id_o, 1u);
+          for (int k = 0; k < 4; ++k) warp_umma_ss(d, ac + 2 * k, bc + 2 * k, id_s, c + k > 0);
+        } else {
+          for (int k = 0; k < rest; ++k) warp_umma_ss(d, ac + 2 * k, bc + 2 * k, id_s, c + k > 0);
         }
-        umma_commit(smem_u32(&b_empty[st]));
-        umma_commit(smem_u32(&b_pv[g]));
-        if (j + 2 < tb) scores(j + 2);             // behind the product that reads these columns' weights
-        if (j + 1 == tb) umma_commit(smem_u32(&b_o[g]));
       }
+      warp_umma_commit(smem_u32(&b_s[g][buf]));
+    };
+    bar_wait(&b_q, 0, abort_flag, p.status);
+    for (int j = 0; j < tiles; ++j) {
+      const int st = j % kStages;
+      if (j < ta || j >= tb) {
+        bar_wait(&b_full[st], (j / kStages) & 1, abort_flag, p.status);
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&b_empty[st]));
+        continue;
+      }
+      if (j == ta) {
+        scores(j);
+        if (j + 1 < tb) scores(j + 1);
+      }
+      const int n = j - ta, buf = n & 1;
+      bar_wait(&b_p[g][buf], (n >> 1) & 1, abort_flag, p.status);
+      __syncwarp();
+      tc_fence_after();
+      const uint32_t b = desc_lo_mn(s_v + st * vs * kSlab, kSlab), pw = t_s + buf * 64;
+#pragma unroll
+      for (int k = 0; k < kTileKeys / 16; ++k) {                              // 16 keys: 2048 bytes of v
+        warp_umma_ts(t_o, pw + k * 8, b + k * 128, id_o, (n > 0 || k > 0) ? 1u : 0u);
+        warp_umma_ts(t_o, pw + 32 + k * 8, b + k * 128, id_o, 1u);
+      }
+      warp_umma_commit(smem_u32(&b_empty[st]));
+      warp_umma_commit(smem_u32(&b_pv[g]));
+      if (j + 2 < tb) scores(j + 2);               // behind the product that reads these columns' weights
+      if (j + 1 == tb) warp_umma_commit(smem_u32(&b_o[g]));
     }
   } else if (warp >= 8) {
     // ---- copies ----
