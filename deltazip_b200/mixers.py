@@ -388,7 +388,8 @@ class LightningSpec:
 
     @classmethod
     def from_dict(cls, d: dict) -> "LightningSpec":
-        spec = cls(int(d["heads"]), int(d["dim"]), int(d["vdim"]), tuple(float(x) for x in d["decay"]))
+        decay = d["decay"] if isinstance(d["decay"], (list, tuple)) else [d["decay"]] * int(d["heads"])
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d["vdim"]), tuple(float(x) for x in decay))
         if len(spec.decay) != spec.heads:
             raise ValueError("one decay per head")
         return spec

@@ -146,14 +146,18 @@ SHAPES = [(3, 56, 8), (6, 96, 16), (16, 512, 64), (20, 64, 24), (40, 128, 8), (1
 @pytest.mark.parametrize("shape", SHAPES)
 @pytest.mark.parametrize("dtype", [F32, F16, BF16])
 def test_latent_attention_kernels(shape, dtype):
+    from deltazip_b200 import ops
     heads, rank, rot = shape
     t = 300 if heads * rank < 3000 else 140
     r = LatentRun(heads, rank, rot, t, dtype, seed=rank, sink=np.random.default_rng(1).normal(size=heads))
     for lo, hi in ((t - 1, t), (0, 1), (63, 65), (100, 116), (0, 40)):
         for splits in (0, 1, 3, 16):
             assert rel(r.run(lo, hi, splits), r.want[lo:hi]) < EXACT[dtype], (lo, hi, splits)
-    r = LatentRun(heads, rank, rot, 70, dtype, seed=rank)                # without a sink
-    assert rel(r.run(60, 70), r.want[60:]) < EXACT[dtype]
+    # without a sink, other page sizes (those that are not a multiple of eight have a kernel of their own)
+    for block in (12, 16, 24, 64, 128):
+        r = LatentRun(heads, rank, rot, 90, dtype, seed=block, block=block)
+        assert rel(r.run(70, 90), r.want[70:]) < EXACT[dtype], block
+    assert ops.read_status() == 0
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
@@ -192,6 +196,20 @@ def test_split_launches_of_changing_batch_size_share_a_workspace():
         want = call(most, 1)
         for n in (most, 1, most, 2, 3, most):
             assert rel(host(call(n, 4)), host(want[:n])) < 1e-2, (name, n)
+
+
+@pytest.mark.parametrize("grow", [False, True])
+def test_latent_attention_with_scores_that_grow_along_the_keys(grow):
+    """The running maximum moves by far more than rounding allows to ignore, in every tile or in none, also
+    where the largest score comes first."""
+    t, heads, rank, rot = 700, 20, 136, 24
+    rng = np.random.default_rng(6)
+    rows, q = rng.normal(size=(t, rank + rot)) * 0.2, np.zeros((t, heads, rank + rot))
+    rows[:, 0] = np.linspace(0, 60, t)[::1 if grow else -1]
+    q[..., 0], q[..., 1:] = 2.0, rng.normal(size=(t, heads, rank + rot - 1)) * 0.1
+    r = LatentRun(heads, rank, rot, t, F16, scale=0.8, rows=rows, q=q, sink=rng.normal(size=heads) * 20)
+    for splits in (1, 4):
+        assert rel(r.run(t - 2, t, splits), r.want[t - 2:]) < EXACT[F16]
 
 
 def test_first_tokens_see_themselves_and_the_sink():
