@@ -13,8 +13,7 @@
 // Roles: warps 0 and 4 softmax (a lane owns a head, a warp half of a tile's keys: scores from TMEM, running
 // maximum, exponentials, weights into shared memory), warps 1 and 3 copies (half of the columns each; TMA,
 // one box per slab and run of rows that lie together in a page), warp 2 MMA issue, warps 8-11 rescaling of
-// the sums (rare: the maximum is moved only when it has grown by more than 2^8) and the output.  All waits
-// are bounded.
+// the sums (rare: the maximum is moved only when it has grown by more than 2^8).  All waits are bounded.
 #include <algorithm>
 #include <numeric>
 
@@ -289,17 +288,17 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       if (lane == 0) mbar_arrive(smem_u32(&b_p[buf]));
     }
     if (tiles > 0) bar_wait(&b_o, 0, abort_flag, p.status);
-    tc_fence_after();
   }
   __syncthreads();
-  if (warp >= 8) {
-    // ---- output ----
+  tc_fence_after();
+  {
+    // ---- output, by all warps ----
     // small loops: this code runs once, and fetching it costs more than running it
     const uint32_t t_o = tmem + kTmemO + ((uint32_t)((warp & 3) * 32) << 16);
     const size_t at = (size_t)row * p.heads + h0;
     const int step = p.splits == 1 ? p.rank : p.splits * partial_row(p.rank);        // from a head to the next
 #pragma unroll 1
-    for (int i = 0; i < tiles_m; ++i) {
+    for (int i = warp >> 2; i < tiles_m; i += kTcThreads / 128) {
       const int c = i * 128 + (warp & 3) * 32 + lane;
       T* out = (T*)p.out + at * p.rank + c;
       float* part = p.partial + (at * p.splits + split) * partial_row(p.rank) + c;

@@ -198,8 +198,12 @@ attention_any_kernel(AttnParams p, int num_seqs) {
 // merged by shuffles, then through shared memory, then -- with splits -- by the last CTA of a
 // (sequence, head group) to arrive at its ticket.  Nothing waits on anything.
 // -------------------------------------------------------------------------------------------------
+// CTAs an SM is to hold: as many as the accumulators' registers allow.
+__host__ __device__ constexpr int decode_ctas(int g, int nk, int nv) {
+  return g * (nk + nv) == 2 ? 4 : g * (nk + nv) == 3 || (g == 2 && nk + nv == 2) ? 3 : g <= 2 || nk + nv == 2 ? 2 : 1;
+}
 template <typename T, int G, int NK, int NV>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, decode_ctas(G, NK, NV))
 window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int* __restrict__ tickets) {
   constexpr int kWarps = 8, VW = NV * 128;
   __shared__ float s_m[kWarps][G], s_l[kWarps][G];
@@ -263,8 +267,8 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
       const int d = (c * 16 + hl) * 8;
       va[c] = vb[c] = make_uint4(0, 0, 0, 0);
       if (d < p.vdim) {
-        va[c] = *reinterpret_cast<const uint4*>(vc + ra * p.v_row + d);
-        vb[c] = *reinterpret_cast<const uint4*>(vc + rb * p.v_row + d);
+        va[c] = *reinterpret_cast<const uint4*>(vc + ra * p.vdim + d);
+        vb[c] = *reinterpret_cast<const uint4*>(vc + rb * p.vdim + d);
       }
     }
     float pa[G], pb[G];
@@ -464,7 +468,7 @@ window_prefill_kernel(AttnParams p, int dimp) {
     } else {
       const size_t s = ring_slot(p, table, t) * p.kv_heads + kvh;
       ks = (const T*)p.k_cache + s * p.dim;
-      vs = (const T*)p.v_cache + s * p.v_row;
+      vs = (const T*)p.v_cache + s * p.vdim;
     }
     T* dk = sk + (buf * kBN + r) * ldk;
     T* dv = sv + (buf * kBN + r) * ldv;

@@ -18,7 +18,7 @@ struct AttnParams {
   int k_off, v_off;                      // columns of `kv` where the key / value parts start
   void* out;                             // [rows, heads * vdim]
   const void* k_cache;                   // [slots, kv_heads, dim]
-  const void* v_cache;                   // [slots, kv_heads, v_row], the first vdim of every v_row
+  const void* v_cache;                   // [slots, kv_heads, vdim]; any-size kernel: the first vdim of every v_row
   int v_row;
   const int* block_tables;               // [sequences, ring_blocks]
   int ring_blocks, block_size;

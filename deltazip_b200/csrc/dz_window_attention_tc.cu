@@ -255,7 +255,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         } else {
           const size_t slot = ring_slot(p, table, key) * p.kv_heads + kvh;
           kp = (const T*)p.k_cache + slot * p.dim;
-          vp = (const T*)p.v_cache + slot * p.v_row;
+          vp = (const T*)p.v_cache + slot * p.vdim;
         }
         for (int e = c; e < p.dim / 8; e += 16) cp_async16_u32(dk + swizzled(r, e, kSlab), kp + e * 8, ok);
         if (c < vcols / 8) cp_async16_u32(dv + swizzled(r, c, kSlab), vp + v0 + c * 8, ok);
