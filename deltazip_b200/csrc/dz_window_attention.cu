@@ -228,8 +228,10 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
   for (int g = 0; g < G; ++g) {
     const int head = kvh * ratio + min(g0 + g, ratio - 1);      // a surplus lane repeats the last head
     bias[g] = p.bias ? p.bias + (size_t)head * p.bias_len : nullptr;
-    m[g] = -INFINITY;
-    l[g] = 0.f;
+    // one half-warp of one split starts with the sink in its sum
+    const bool sink = p.sink && split == 0 && threadIdx.x < 16;
+    m[g] = sink ? p.sink[head] : -INFINITY;
+    l[g] = sink ? 1.f : 0.f;
 #pragma unroll
     for (int c = 0; c < NK; ++c) {
       const int d = (c * 16 + hl) * 8;
@@ -364,11 +366,6 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
     }
     const int head = kvh * ratio + g0 + g;
     if (splits == 1) {
-      if (p.sink) {
-        const float sk = p.sink[head], top = fmaxf(mm, sk), c = __expf(mm - top);
-        a *= c;
-        ll = ll * c + __expf(sk - top);
-      }
       ((T*)p.out)[((size_t)seq * p.heads + head) * p.vdim + d] = Cvt<T>::from(a / ll);
     } else {
       float* pp = partial + (((size_t)seq * p.heads + head) * splits + split) * (p.vdim + 2);
@@ -392,8 +389,7 @@ window_decode_kernel(AttnParams p, int splits, float* __restrict__ partial, int*
     const float* pp = partial + ((size_t)seq * p.heads + head) * splits * w;
     float mm = -INFINITY;
     for (int s = 0; s < splits; ++s) mm = fmaxf(mm, __ldcg(pp + s * w + p.vdim));
-    if (p.sink) mm = fmaxf(mm, p.sink[head]);
-    float ll = p.sink ? __expf(p.sink[head] - mm) : 0.f, a = 0.f;
+    float ll = 0.f, a = 0.f;
     for (int s = 0; s < splits; ++s) {
       const float ms = __ldcg(pp + s * w + p.vdim);
       const float c = ms == -INFINITY ? 0.f : __expf(ms - mm);
