@@ -198,9 +198,9 @@ attention_any_kernel(AttnParams p, int num_seqs) {
 // merged by shuffles, then through shared memory, then -- with splits -- by the last CTA of a
 // (sequence, head group) to arrive at its ticket.  Nothing waits on anything.
 // -------------------------------------------------------------------------------------------------
-// CTAs an SM is to hold: as many as the accumulators' registers allow.
+// CTAs an SM is to hold where the compiler would take registers for fewer; 0: as it likes.
 __host__ __device__ constexpr int decode_ctas(int g, int nk, int nv) {
-  return g * (nk + nv) == 2 ? 4 : g * (nk + nv) == 3 || (g == 2 && nk + nv == 2) ? 3 : g <= 2 || nk + nv == 2 ? 2 : 1;
+  return g != 2 ? 0 : nk + nv == 2 ? 3 : nk + nv == 4 ? 2 : 0;
 }
 template <typename T, int G, int NK, int NV>
 __global__ void __launch_bounds__(256, decode_ctas(G, NK, NV))
